@@ -209,8 +209,8 @@ class CacheManager:
             w = g.need.window
             if not w:
                 continue
-            # the next query sits at position >= n_processed and sees keys > position - w
-            first_visible = max(0, n_processed - w + 1)
+            # the next query sits at position >= n_processed
+            first_visible = g.need.first_visible(n_processed)
             full_pages_behind = min(first_visible // self.page_size, len(rc.tables[g.index]))
             lo = min(self.kept_pages(g.index), full_pages_behind) + rc.released[g.index]
             if full_pages_behind > lo:

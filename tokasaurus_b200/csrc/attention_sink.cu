@@ -45,7 +45,15 @@
 // keep_first: with a window, the first keep_first positions of a request stay visible to every later query
 // (position i sees j if j <= i and (i - j < window or j < keep_first)).
 //
-// Compile with -DTKB_QK=<query/key size> -DTKB_VD=<value size> [-DTKB_SIGMOID=1] [-DTKB_MAPS=2].
+// chunk: the sequence is cut into chunks of so many positions, counted from position 0; a query sees the keys of its own
+// chunk only (position i sees j <= i with i / chunk == j / chunk).
+//
+// A bias by distance, chosen at compile time (-DTKB_DIST=1): head_slope (float32 [heads]) times the distance i - j comes
+// off the score, after scale and cap.
+//
+// Outputs go to rows of out_stride values, multiplied by out_scale (a mixer beside another writes its share of a wider row).
+//
+// Compile with -DTKB_QK=<query/key size> -DTKB_VD=<value size> [-DTKB_SIGMOID=1] [-DTKB_MAPS=2] [-DTKB_DIST=1].
 #include "common.cuh"
 #include <float.h>
 #include <type_traits>
@@ -59,6 +67,9 @@ static_assert(TKB_QK >= 1 && TKB_QK <= 512 && TKB_VD >= 1 && TKB_VD <= 512, "hea
 #endif
 #ifndef TKB_MAPS
 #define TKB_MAPS 1
+#endif
+#ifndef TKB_DIST
+#define TKB_DIST 0
 #endif
 static_assert(TKB_MAPS >= 1 && TKB_MAPS <= 4, "one to four attention maps a head");
 
@@ -74,6 +85,13 @@ constexpr int ROW = KW + VD;
 constexpr int WARPS = 4;
 constexpr int DPL = (VD + 31) / 32;
 constexpr bool SIGMOID = TKB_SIGMOID != 0;
+constexpr bool DIST = TKB_DIST != 0;
+
+// The first key that a query at position p sees (kept first positions aside).
+__device__ __forceinline__ int first_key(int p, int window, int chunk) {
+  const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+  return chunk > 0 ? max(lo, p - p % chunk) : lo;
+}
 
 template <typename T>
 __device__ __forceinline__ float dot_key(const T* __restrict__ k, const float* __restrict__ q) {
@@ -186,8 +204,9 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
                       const int* __restrict__ token_seq, const int* __restrict__ positions,
                       const int* __restrict__ page_indptr, const int* __restrict__ page_ids,
                       const int* __restrict__ rows, const float* __restrict__ sinks, int nh, int nkv, int page_size,
-                      float scale, float softcap, int window, int keep_first, int num_pages, int* __restrict__ status,
-                      const float* __restrict__ head_scale, const float* __restrict__ head_bias) {
+                      float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
+                      int* __restrict__ status, const float* __restrict__ head_scale, const float* __restrict__ head_bias,
+                      const float* __restrict__ head_slope, int out_stride, float out_scale) {
   using TO = typename OutOf<T>::type;
   __shared__ float qs[WARPS][QK];
   trigger_dependents();
@@ -200,8 +219,7 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
   const int group = nh / nkv;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int* table = page_ids + page_indptr[s];
-  int lo = 0;
-  if (window > 0 && p - window + 1 > 0) lo = p - window + 1;
+  const int lo = first_key(p, window, chunk);
   // the positions kept in sight before the window: [0, kept)
   const int kept = (window > 0 && keep_first > 0) ? min(keep_first, lo) : 0;
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
@@ -214,6 +232,7 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
     __syncwarp();
 
     const float hscale = scale * (head_scale ? head_scale[h] : 1.f), hbias = head_bias ? head_bias[h] : 0.f;
+    const float slope = DIST && head_slope ? head_slope[h] : 0.f;
     // the sink opens the running softmax: maximum sink, sum exp(sink - sink) = 1, nothing accumulated
     float m = sinks ? sinks[h] : -FLT_MAX;
     float l = sinks ? 1.f : 0.f;
@@ -236,6 +255,7 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
             sc = dot_key<T>(cache + rowoff + koff, qs[warp]) * hscale;
             if (softcap > 0.f) sc = softcap * tanhf(sc * inv_cap);
             sc += hbias;
+            if (DIST) sc = fmaf(slope, (float)(j - p), sc);
             counted = true;
           }
         }
@@ -265,8 +285,8 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
         }
       }
     }
-    const float inv_l = SIGMOID ? 1.f : (l > 0.f ? 1.f / l : 0.f);
-    TO* orow = out + ((size_t)blockIdx.x * nh * MAPS + h) * VD;
+    const float inv_l = (SIGMOID ? 1.f : (l > 0.f ? 1.f / l : 0.f)) * out_scale;
+    TO* orow = out + (size_t)blockIdx.x * out_stride + (size_t)h * VD;
 #pragma unroll
     for (int i = 0; i < DPL; i++) {
       const int d = lane + 32 * i;
@@ -326,15 +346,17 @@ int prep_launch(const float* qkv, int stride, const float* bias, int unit_norm, 
 template <typename T>
 int attn_launch(const void* q, void* out, const void* cache, const int* token_seq, const int* positions,
                 const int* page_indptr, const int* page_ids, const int* rows, int n_rows, const float* sinks, int nh,
-                int nkv, int page_size, float scale, float softcap, int window, int keep_first, int num_pages,
-                int* status, const float* head_scale, const float* head_bias, cudaStream_t st) {
+                int nkv, int page_size, float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
+                int* status, const float* head_scale, const float* head_bias, const float* head_slope, int out_stride,
+                float out_scale, cudaStream_t st) {
   if (n_rows <= 0) return 0;
-  if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || keep_first < 0) return -2;
+  if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || keep_first < 0 || (head_slope != nullptr && !DIST)) return -2;
+  if (out_stride < nh * MAPS * VD) return -2;
   if (nkv > 65535) return -3;
   return launch_pdl(attn_sink_simt_kernel<T>, dim3(n_rows, nkv), dim3(WARPS * 32), 0, st, (const T*)q,
                     (typename OutOf<T>::type*)out, (const T*)cache, token_seq, positions, page_indptr, page_ids, rows,
-                    sinks, nh, nkv, page_size, scale, softcap, window, keep_first, num_pages, status, head_scale,
-                    head_bias);
+                    sinks, nh, nkv, page_size, scale, softcap, window, keep_first, chunk, num_pages, status, head_scale,
+                    head_bias, head_slope, out_stride, out_scale);
 }
 
 }  // namespace
@@ -354,11 +376,12 @@ int attn_launch(const void* q, void* out, const void* cache, const int* token_se
                                           const int* positions, const int* page_indptr, const int* page_ids,          \
                                           const int* rows, int n_rows, const float* sinks, int nh, int nkv,           \
                                           int page_size, float scale, float softcap, int window, int keep_first,      \
-                                          int num_pages, int* status, const float* head_scale,                        \
-                                          const float* head_bias, void* st) {                                         \
+                                          int chunk, int num_pages, int* status, const float* head_scale,             \
+                                          const float* head_bias, const float* head_slope, int out_stride,            \
+                                          float out_scale, void* st) {                                                \
     return attn_launch<T>(q, out, cache, token_seq, positions, page_indptr, page_ids, rows, n_rows, sinks, nh, nkv,   \
-                          page_size, scale, softcap, window, keep_first, num_pages, status, head_scale, head_bias,    \
-                          (cudaStream_t)st);                                                                          \
+                          page_size, scale, softcap, window, keep_first, chunk, num_pages, status, head_scale,        \
+                          head_bias, head_slope, out_stride, out_scale, (cudaStream_t)st);                                                                          \
   }                                                                                                                   \
   TKB_EXPORT int tkb_diff_combine_##SUF(const float* a, const float* lambda, float eps, float mult,                   \
                                         const float* gate, int gate_stride, int gate_off, const int* rows, void* out, \
@@ -465,12 +488,13 @@ __device__ __forceinline__ void stage_tile(bf16* buf, const bf16* __restrict__ c
 // One warp, 16 rows, NT groups of 8 keys that start at row `kr0` of the staged tile (key index key0): scores, running
 // softmax, and the weighted sum of values.  lim_lo / lim_hi: the keys each of the thread's two rows may see; keys
 // below `keep` are seen from below lim_lo too (the first positions that a window keeps).  koff: where the map's key
-// starts in a staged row.
+// starts in a staged row.  slope2, qpos (DIST): the rows' slopes in units of log2, and their positions.
 // MASKED false: every key of the span is seen by every row (the caller has checked), no limit is looked at.
 template <int NT, bool MASKED>
 __device__ __forceinline__ void attend(const bf16* buf, int kr0, int key0, const uint32_t (&qf)[KSTEPS][4], float (&o)[VT][4],
                                        float (&m)[2], float (&l)[2], const int (&lim_lo)[2], const int (&lim_hi)[2],
-                                       const ScoreMap (&sm)[2], int lane, int koff = 0, int keep = 0) {
+                                       const ScoreMap (&sm)[2], int lane, int koff, int keep, const float (&slope2)[2],
+                                       const int (&qpos)[2]) {
   const int g = lane >> 2, t = lane & 3;
   float sc[NT][4];
 #pragma unroll
@@ -504,7 +528,9 @@ __device__ __forceinline__ void attend(const bf16* buf, int kr0, int key0, const
       for (int nt = 0; nt < NT; nt++)
 #pragma unroll
         for (int e = 0; e < 2; e++) {
-          float v = sigmoid2(mapped_score(sc[nt][h * 2 + e], sm[h]));
+          float v = mapped_score(sc[nt][h * 2 + e], sm[h]);
+          if (DIST) v = fmaf(slope2[h], (float)(key0 + nt * 8 + 2 * t + e - qpos[h]), v);
+          v = sigmoid2(v);
           if (MASKED) {
             const int key = key0 + nt * 8 + 2 * t + e;
             if ((key < lim_lo[h] && key >= keep) || key > lim_hi[h]) v = 0.f;
@@ -521,6 +547,7 @@ __device__ __forceinline__ void attend(const bf16* buf, int kr0, int key0, const
 #pragma unroll
       for (int e = 0; e < 2; e++) {
         float v = mapped_score(sc[nt][h * 2 + e], sm[h]);
+        if (DIST) v = fmaf(slope2[h], (float)(key0 + nt * 8 + 2 * t + e - qpos[h]), v);
         if (MASKED) {
           const int key = key0 + nt * 8 + 2 * t + e;
           if ((key < lim_lo[h] && key >= keep) || key > lim_hi[h]) v = -INFINITY;
@@ -576,8 +603,9 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
                        const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
                        const int* __restrict__ seq_kv_len, const int* __restrict__ page_indptr,
                        const int* __restrict__ page_ids, int n_seqs, const float* __restrict__ sinks, int nh, int nkv,
-                       int ps, float scale, float softcap, int window, int keep_first, int num_pages, int* __restrict__ status,
-                       const float* __restrict__ head_scale, const float* __restrict__ head_bias) {
+                       int ps, float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
+                       int* __restrict__ status, const float* __restrict__ head_scale, const float* __restrict__ head_bias,
+                       const float* __restrict__ head_slope, int out_stride, float out_scale) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* bufs = reinterpret_cast<bf16*>(smem_raw);
   trigger_dependents();
@@ -602,16 +630,19 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
   const int* table = page_ids + page_indptr[s];
   const ScoreMap sm1 = score_map(scale * (head_scale ? head_scale[h] : 1.f), softcap, head_bias ? head_bias[h] : 0.f);
   const ScoreMap sm[2] = {sm1, sm1};
+  const float slope1 = DIST && head_slope ? head_slope[h] * LOG2E : 0.f;
+  const float slope2[2] = {slope1, slope1};
 
   uint32_t qf[KSTEPS][4];
-  int lim_lo[2], lim_hi[2];
+  int lim_lo[2], lim_hi[2], qpos[2];
 #pragma unroll
   for (int hh = 0; hh < 2; hh++) {
     const int r = warp * 16 + g + hh * 8;
     const bool live = r < rows;
     const int p = pos0 + r0 + r;
+    qpos[hh] = p;
     lim_hi[hh] = live ? p : -1;
-    lim_lo[hh] = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+    lim_lo[hh] = first_key(p, window, chunk);
     const bf16* qrow = q + ((size_t)(start + r0 + (live ? r : 0)) * nhm + h) * QK;
 #pragma unroll
     for (int ks = 0; ks < KSTEPS; ks++) {
@@ -629,7 +660,7 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
   for (int vt = 0; vt < VT; vt++) o[vt][0] = o[vt][1] = o[vt][2] = o[vt][3] = 0.f;
 
   const int p_first = pos0 + r0, p_last = pos0 + r0 + rows - 1;
-  const int k_lo = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+  const int k_lo = first_key(p_first, window, chunk);
   // the first positions that the window keeps in sight: [0, kept) lies before every row's window and is staged in
   // tiles of its own, which come first; kept positions from k_lo on arrive with the window's tiles
   const int keep = window > 0 ? keep_first : 0;
@@ -641,9 +672,9 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
   auto tile_last = [&](int it) { return it < keep_tiles ? kept - 1 : p_last; };
   // the keys this warp's rows can see within the window's tiles: [w_lo, w_hi]
   const int w_first = pos0 + r0 + warp * 16;
-  const int w_lo = keep > k_lo ? k_lo : ((window > 0 && w_first - window + 1 > 0) ? w_first - window + 1 : 0);
+  const int w_lo = keep > k_lo ? k_lo : first_key(w_first, window, chunk);
   const int w_hi = min(p_last, w_first + 15);
-  const int w_last_lo = (window > 0 && w_first + 15 - window + 1 > 0) ? w_first + 15 - window + 1 : 0;  // the last row's
+  const int w_last_lo = first_key(w_first + 15, window, chunk);  // the last row's
   bool bad = false;
   stage_tile(bufs, cache, table, tile_key0(0), tile_first(0), tile_last(0), kvh, nkv, ps, num_pages, bad, tid);
   cp_async_commit();
@@ -663,14 +694,14 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
       // kept positions: every live row sees [0, kept), nothing beyond in this tile
       if (warp * 16 < rows) {
         const int kl[2] = {0, 0}, kh[2] = {lim_hi[0] < 0 ? -1 : kept - 1, lim_hi[1] < 0 ? -1 : kept - 1};
-        attend<8, true>(cur, 0, key0, qf, o, m, l, kl, kh, sm, lane, koff, 0);
+        attend<8, true>(cur, 0, key0, qf, o, m, l, kl, kh, sm, lane, koff, 0, slope2, qpos);
       }
     } else if (warp * 16 < rows && key0 <= w_hi && key0 + KT - 1 >= w_lo) {  // warp-uniform: some row of the warp sees some key
       // all 16 rows live and the whole tile inside every row's window and before the warp's first query: no masks
       if (warp * 16 + 16 <= rows && key0 + KT - 1 <= w_first && key0 >= w_last_lo)
-        attend<8, false>(cur, 0, key0, qf, o, m, l, lim_lo, lim_hi, sm, lane, koff, keep);
+        attend<8, false>(cur, 0, key0, qf, o, m, l, lim_lo, lim_hi, sm, lane, koff, keep, slope2, qpos);
       else
-        attend<8, true>(cur, 0, key0, qf, o, m, l, lim_lo, lim_hi, sm, lane, koff, keep);
+        attend<8, true>(cur, 0, key0, qf, o, m, l, lim_lo, lim_hi, sm, lane, koff, keep, slope2, qpos);
     }
     __syncthreads();  // the buffer is free for the tile after next
   }
@@ -681,8 +712,8 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
     l[hh] += __shfl_xor_sync(0xffffffffu, l[hh], 2);
     const int r = warp * 16 + g + hh * 8;
     if (r < rows) {
-      const float inv = l[hh] > 0.f ? 1.f / l[hh] : 0.f;
-      auto* orow = out + ((size_t)(start + r0 + r) * nhm + h) * VD + 2 * t;
+      const float inv = l[hh] > 0.f ? out_scale / l[hh] : 0.f;
+      auto* orow = out + (size_t)(start + r0 + r) * out_stride + (size_t)h * VD + 2 * t;
 #pragma unroll
       for (int vt = 0; vt < VT; vt++) {
         if constexpr (MAPS > 1)
@@ -704,9 +735,10 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
                         const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
                         const int* __restrict__ seq_kv_len, const int* __restrict__ page_indptr,
                         const int* __restrict__ page_ids, const float* __restrict__ sinks, int nh, int nkv, int head_tiles,
-                        int ps, float scale, float softcap, int window, int keep_first, int num_pages,
+                        int ps, float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
                         int* __restrict__ status, float* __restrict__ part, const float* __restrict__ head_scale,
-                        const float* __restrict__ head_bias) {
+                        const float* __restrict__ head_bias, const float* __restrict__ head_slope, int out_stride,
+                        float out_scale) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* bufs = reinterpret_cast<bf16*>(smem_raw);
   trigger_dependents();
@@ -723,7 +755,9 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
   const int p = seq_kv_len[s] - 1;
   const int* table = page_ids + page_indptr[s];
   ScoreMap sm[2];
-  const int k_lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+  float slope2[2];
+  const int qpos[2] = {p, p};
+  const int k_lo = first_key(p, window, chunk);
 
   uint32_t qf[KSTEPS][4];
   float m[2], l[2];
@@ -739,6 +773,7 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
       qf[ks][hh + 2] = live ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 8 + 2 * t) : 0u;
     }
     sm[hh] = score_map(scale * (head_scale ? head_scale[head] : 1.f), softcap, head_bias ? head_bias[head] : 0.f);
+    slope2[hh] = DIST && head_slope ? head_slope[head] * LOG2E : 0.f;
     // (the sigmoid form: every share has maximum 0, and ONE share carries the sum 1, so the merges below only add)
     m[hh] = SIGMOID ? 0.f : (sinks ? sinks[head] * LOG2E : NEG_BIG);
     l[hh] = ((SIGMOID || sinks) && split == 0 && wsub == 0 && t == 0) ? 1.f : 0.f;  // the sink counts once: in one warp's sums
@@ -777,7 +812,7 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
     const int last = tile_last(it0 + it);
     if (key0 <= last) {
       const int tl[2] = {tile_first(it0 + it), tile_first(it0 + it)}, th[2] = {last, last};
-      attend<KPW / 8, true>(cur, wsub * KPW, key0, qf, o, m, l, tl, th, sm, lane, koff, 0);
+      attend<KPW / 8, true>(cur, wsub * KPW, key0, qf, o, m, l, tl, th, sm, lane, koff, 0, slope2, qpos);
     }
     __syncthreads();
   }
@@ -820,7 +855,7 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
     }
     const int head = (kvh * group + g0 + r) * MAPS + mp;
     if (splits == 1) {
-      out[((size_t)tok * nhm + head) * VD + d] = from_float<OutOf<bf16>::type>(ll > 0.f ? acc / ll : 0.f);
+      out[(size_t)tok * out_stride + (size_t)head * VD + d] = from_float<OutOf<bf16>::type>(ll > 0.f ? acc / ll * out_scale : 0.f);
     } else {  // this split's share: sums relative to its own maximum, for attn_sink_merge
       float* pr = part + (((size_t)s * nhm + head) * splits + split) * (VD + 2);
       pr[d] = acc;
@@ -835,7 +870,7 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
 // The splits of every single-token request put together: grid (request row, query head).
 __global__ void attn_sink_merge_kernel(const float* __restrict__ part, OutOf<bf16>::type* __restrict__ out,
                                        const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len, int nh,
-                                       int splits) {
+                                       int splits, int out_stride, float out_scale) {
   trigger_dependents();
   grid_dependency_wait();
   const int s = blockIdx.x, head = blockIdx.y;
@@ -845,11 +880,11 @@ __global__ void attn_sink_merge_kernel(const float* __restrict__ part, OutOf<bf1
   for (int z = 0; z < splits; z++) mm = fmaxf(mm, pr[z * (VD + 2) + VD]);
   float ll = 0.f;
   for (int z = 0; z < splits; z++) ll += exp2f(pr[z * (VD + 2) + VD] - mm) * pr[z * (VD + 2) + VD + 1];
-  const float inv = ll > 0.f ? 1.f / ll : 0.f;
+  const float inv = ll > 0.f ? out_scale / ll : 0.f;
   for (int d = threadIdx.x; d < VD; d += blockDim.x) {
     float acc = 0.f;
     for (int z = 0; z < splits; z++) acc += exp2f(pr[z * (VD + 2) + VD] - mm) * pr[z * (VD + 2) + d];
-    out[((size_t)seq_q_start[s] * nh + head) * VD + d] = from_float<OutOf<bf16>::type>(acc * inv);
+    out[(size_t)seq_q_start[s] * out_stride + (size_t)head * VD + d] = from_float<OutOf<bf16>::type>(acc * inv);
   }
 }
 
@@ -863,11 +898,14 @@ TKB_EXPORT int tkb_attn_sink_tc_bf16(const void* q, void* out, const void* cache
                                      const int* seq_q_len, const int* seq_kv_len, const int* page_indptr,
                                      const int* page_ids, int n_tokens, int n_seqs, int portions, int singles,
                                      const float* sinks, int nh, int nkv, int page_size, float scale, float softcap,
-                                     int window, int keep_first, int num_pages, int* status, float* part, int splits,
-                                     const float* head_scale, const float* head_bias, void* st) {
+                                     int window, int keep_first, int chunk, int num_pages, int* status, float* part,
+                                     int splits, const float* head_scale, const float* head_bias,
+                                     const float* head_slope, int out_stride, float out_scale, void* st) {
   using TO = OutOf<bf16>::type;
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
-  if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || keep_first < 0) return -2;
+  if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || keep_first < 0 || (head_slope != nullptr && !DIST)) return -2;
+  // (the portions' kernel stores pairs of values)
+  if (out_stride < nh * MAPS * VD || (out_stride & 1) || (((uintptr_t)out) & 7)) return -2;
   const int head_tiles = (nh / nkv + 15) / 16;
   if (nh * MAPS > 65535 || nkv * head_tiles > 65535) return -3;
   if (TC_SMEM > 48 * 1024) {
@@ -883,18 +921,19 @@ TKB_EXPORT int tkb_attn_sink_tc_bf16(const void* q, void* out, const void* cache
     rc = launch_pdl(attn_sink_single_kernel, dim3(n_seqs, nkv * head_tiles, splits), dim3(128), TC_SMEM,
                     (cudaStream_t)st, (const bf16*)q, (TO*)out, (const bf16*)cache, seq_q_start, seq_q_len, seq_kv_len,
                     page_indptr, page_ids, sinks, nh, nkv, head_tiles, page_size, scale, softcap, window, keep_first,
-                    num_pages, status, part, head_scale, head_bias);
+                    chunk, num_pages, status, part, head_scale, head_bias, head_slope, out_stride, out_scale);
     if (rc == 0 && splits > 1)
       rc = launch_pdl(attn_sink_merge_kernel, dim3(n_seqs, nh * MAPS), dim3(VD >= 128 ? 128 : 64), 0, (cudaStream_t)st,
-                      (const float*)part, (TO*)out, seq_q_start, seq_q_len, nh * MAPS, splits);
+                      (const float*)part, (TO*)out, seq_q_start, seq_q_len, nh * MAPS, splits,
+                      out_stride, out_scale);
   }
   if (rc != 0 || !portions) return rc;
   const int tiles = n_tokens / KT + n_seqs;  // no step of this shape has more 64-query tiles
   if (tiles > 65535) return -3;
   return launch_pdl(attn_sink_tiles_kernel, dim3(nh * MAPS, tiles), dim3(128), TC_SMEM, (cudaStream_t)st, (const bf16*)q,
                     (TO*)out, (const bf16*)cache, seq_q_start, seq_q_len, seq_kv_len, page_indptr, page_ids, n_seqs,
-                    sinks, nh, nkv, page_size, scale, softcap, window, keep_first, num_pages, status, head_scale,
-                    head_bias);
+                    sinks, nh, nkv, page_size, scale, softcap, window, keep_first, chunk, num_pages, status, head_scale,
+                    head_bias, head_slope, out_stride, out_scale);
 }
 #endif  // tensor-core sizes
 TKB_EXPORT int tkb_attn_sink_has_tc() {

@@ -10,7 +10,11 @@
 //     time with bias and SiLU, dt_t = softplus(dt_raw + dt_bias).
 //   * gated linear attention: a DIFFERENT decay for every key channel, S_t = diag(f_t) S_(t-1) + k_t v_t^T, with
 //     f_t = sigmoid(A2 (A1 h_t) + b)^(1/tau) made beforehand for all tokens (gla_gates, which also scales q);
-//   * retention: a_t = lambda_head, q and k rotated by position and k scaled beforehand (rotate_scale).
+//   * retention: a_t = lambda_head, q and k rotated by position and k scaled beforehand (rotate_scale);
+//   * matrix memory: a_t and c_t from two exponential gates a head and token, kept in range by a running maximum
+//     (memory_gates); a normaliser n_t = a_t n_(t-1) + c_t k_t runs along as one more column of S whose values are all 1
+//     (`ones`: the state then holds vdim + 1 columns a head), and its n_t . q_t leaves beside the outputs for the head
+//     norm that divides by it (memory_norm).
 // Everything here is float32: projections arrive as float32 rows, the state lives in the request's slot as S^T,
 // state[slot][head][vdim][dim], and the outputs leave as float32 rows for the norm that follows.
 //
@@ -131,7 +135,9 @@ __global__ void silu_cols_kernel(float* __restrict__ x, int stride, int ncols) {
 constexpr int QROW = LANES * DPT;
 
 // VEC: a decay for every key channel, fvec [T, heads * dim] rows of f_stride floats, staged beside q and k.
-template <bool VEC>
+// ONES: behind a head's vdim columns the state holds one more, whose value is 1 at every token; the last block of a head
+// (blockIdx.z) walks it beside its own, and its output goes to ones_out [T, heads].
+template <bool VEC, bool ONES>
 __global__ void __launch_bounds__(1024)
 decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __restrict__ k, int k_stride, int qk_div,
                   const float* __restrict__ fvec, int f_stride,
@@ -139,9 +145,10 @@ decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __rest
                   const float* __restrict__ decay_head, const float* __restrict__ skip, float* __restrict__ state,
                   long long slot_stride, float* __restrict__ out, const int* __restrict__ seq_slot,
                   const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len, int heads, int dim, int vdim,
-                  int write_state, int cols_per_block, int vec_qk, int vec_v, int vec_s, int chunk) {
+                  int write_state, int cols_per_block, int vec_qk, int vec_v, int vec_s, int chunk,
+                  float* __restrict__ ones_out) {
   extern __shared__ __align__(16) float smem[];
-  const int cols = min(cols_per_block, vdim);
+  const int cols = min(cols_per_block, vdim) + (ONES ? 1 : 0);
   const int cols4 = (cols + 3) & ~3;
   constexpr int NQ = VEC ? 3 : 2;  // staged rows of QROW floats a token: q, k (and the decays)
   const int buf_floats = chunk * (NQ * QROW + cols4 + 2);
@@ -153,16 +160,18 @@ decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __rest
   const int start = seq_q_start[s];
   const int tid = threadIdx.x, lane = tid & (LANES - 1);
   const int col_begin = blockIdx.z * cols_per_block;
-  const int col_end = min(vdim, col_begin + cols_per_block);
-  if (col_begin >= col_end) return;
-  const int ncols = col_end - col_begin;
+  const int v_end = min(vdim, col_begin + cols_per_block);
+  if (col_begin >= v_end) return;
+  const int nv = v_end - col_begin;  // columns with values of their own
+  const int ncols = nv + (ONES && v_end == vdim ? 1 : 0);
+  const int col_end = col_begin + ncols;
   const int lc = tid / LANES;  // this thread's column within the block
   const int j = col_begin + lc;
   // dims beyond `dim` of the last lanes are read: zero the buffers once if there are any (the copies never touch them)
   if (dim < LANES * DPT)
     for (int idx = tid; idx < 2 * buf_floats; idx += blockDim.x) smem[idx] = 0.f;
   grid_dependency_wait();
-  float* st = state + (size_t)seq_slot[s] * slot_stride + (size_t)head * vdim * dim;
+  float* st = state + (size_t)seq_slot[s] * slot_stride + (size_t)head * (vdim + (ONES ? 1 : 0)) * dim;
 
   float S[DPT];
   if (vec_s) {
@@ -212,15 +221,15 @@ decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __rest
         if (VEC) cp_async4(fs + t * QROW + d, fh + (size_t)(start + t0 + t) * f_stride + d);
       }
     }
-    if (vec_v && (ncols & 3) == 0) {
-      const int c4n = ncols >> 2;
+    if (vec_v && (nv & 3) == 0) {
+      const int c4n = nv >> 2;
       for (int idx = tid; idx < nt * c4n; idx += blockDim.x) {
         const int t = idx / c4n, jj = (idx - t * c4n) * 4;
         cp_async16(vs + t * cols4 + jj, vh + (size_t)(start + t0 + t) * v_stride + jj);
       }
     } else {
-      for (int idx = tid; idx < nt * ncols; idx += blockDim.x) {
-        const int t = idx / ncols, jj = idx - t * ncols;
+      for (int idx = tid; idx < nt * nv; idx += blockDim.x) {
+        const int t = idx / nv, jj = idx - t * nv;
         cp_async4(vs + t * cols4 + jj, vh + (size_t)(start + t0 + t) * v_stride + jj);
       }
     }
@@ -251,13 +260,15 @@ decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __rest
     const float* as = vs + chunk * cols4;
     const float* cs = as + chunk;
     float* mine = os + (lc * LANES + lane) * orow;
+    // (a warp that owns no column, where the last block alone has one more than the others, walks over nothing)
+    const int walk = ONES && (tid & ~31) / LANES >= ncols ? 0 : nt;
 #pragma unroll 4
-    for (int t = 0; t < nt; t++) {
+    for (int t = 0; t < walk; t++) {
       const float a = dt_dec ? as[t] : a_const, ck = dt_dec ? cs[t] : 1.f;
       const float4* q4 = reinterpret_cast<const float4*>(qs + t * QROW) + lane;
       const float4* k4 = reinterpret_cast<const float4*>(ks + t * QROW) + lane;
       const float4* f4 = reinterpret_cast<const float4*>(fs + t * QROW) + lane;
-      const float vj = lc < ncols ? vs[t * cols4 + lc] : 0.f;
+      const float vj = lc < nv ? vs[t * cols4 + lc] : (ONES && lc < ncols ? 1.f : 0.f);
       const float cv = ck * vj;
       float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
 #pragma unroll
@@ -288,7 +299,10 @@ decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __rest
     __syncwarp();  // a column's lanes are one warp, or part of one: its shares are all there
     // add the shares up: the lanes of a column split the chunk's tokens among them
     if (lc < ncols) {
-      float* col_out = out + (size_t)(start + t0) * heads * vdim + (size_t)head * vdim + j;
+      const bool one = ONES && lc == nv;
+      const int per_token = one ? heads : heads * vdim;
+      float* col_out = one ? ones_out + (size_t)(start + t0) * heads + head
+                           : out + (size_t)(start + t0) * heads * vdim + (size_t)head * vdim + j;
       const float* shares = os + (size_t)lc * LANES * orow;
       if (LANES == 32 && chunk == 16) {
         const int t = lane & 15, l0 = (lane >> 4) * 16;
@@ -296,13 +310,13 @@ decay_walk_kernel(const float* __restrict__ q, int q_stride, const float* __rest
 #pragma unroll
         for (int l = 0; l < 16; l++) sum += shares[(l0 + l) * orow + t];
         sum += __shfl_xor_sync(0xffffffffu, sum, 16);
-        if (lane < 16 && t < nt) col_out[(size_t)t * heads * vdim] = sum;
+        if (lane < 16 && t < nt) col_out[(size_t)t * per_token] = sum;
       } else {
         for (int t = lane; t < nt; t += LANES) {
           float sum = 0.f;
 #pragma unroll
           for (int l = 0; l < LANES; l++) sum += shares[l * orow + t];
-          col_out[(size_t)t * heads * vdim] = sum;
+          col_out[(size_t)t * per_token] = sum;
         }
       }
     }
@@ -331,7 +345,7 @@ int walk_launch(const float* q, int q_stride, const float* k, int k_stride, int 
                 const float* v, int v_stride,
                 const float* dt_dec, const float* decay_head, const float* skip, float* state, long long slot_stride,
                 float* out, const int* seq_slot, const int* seq_q_start, const int* seq_q_len, int n_seqs, int n_tokens,
-                int heads, int dim, int vdim, int write_state, cudaStream_t st) {
+                int heads, int dim, int vdim, int write_state, float* ones_out, cudaStream_t st) {
   if (n_seqs <= 0 || n_tokens <= 0) return 0;
   if (dim <= 0 || dim > DPT * LANES || vdim <= 0 || heads <= 0 || qk_div <= 0) return -2;
   if (heads > 65535) return -3;
@@ -343,14 +357,15 @@ int walk_launch(const float* q, int q_stride, const float* k, int k_stride, int 
   if (cols_per_block > vdim) cols_per_block = vdim;
   const int splits = (vdim + cols_per_block - 1) / cols_per_block;
   if (splits > 65535) return -3;
-  const int threads = ((cols_per_block * LANES + 31) / 32) * 32;
-  const int cols4 = (cols_per_block + 3) & ~3;
+  const int cols = cols_per_block + (ones_out != nullptr ? 1 : 0);
+  const int threads = ((cols * LANES + 31) / 32) * 32;
+  const int cols4 = (cols + 3) & ~3;
   const int nq = fvec != nullptr ? 3 : 2;
-  const size_t smem = (size_t)(2 * chunk * (nq * QROW + cols4 + 2) + cols_per_block * LANES * (chunk + 1)) * sizeof(float);
+  const size_t smem = (size_t)(2 * chunk * (nq * QROW + cols4 + 2) + threads * (chunk + 1)) * sizeof(float);  // (threads past the last column write shares too)
+  auto kernel = fvec != nullptr ? decay_walk_kernel<true, false>
+                                : (ones_out != nullptr ? decay_walk_kernel<false, true> : decay_walk_kernel<false, false>);
   if (smem > 48 * 1024) {
-    cudaError_t e = fvec != nullptr
-                        ? cudaFuncSetAttribute(decay_walk_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
-                        : cudaFuncSetAttribute(decay_walk_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
@@ -361,14 +376,9 @@ int walk_launch(const float* q, int q_stride, const float* k, int k_stride, int 
   // An ordinary launch, not a programmatic one: blocks that come onto the SMs while the kernel ahead still holds some of
   // them are placed where room happens to be, several to an SM, and this kernel's few long-lived blocks then run on a
   // part of the GPU (measured: 0.84 ms instead of 0.36 ms for 2,048 tokens of 16 heads).
-  if (fvec != nullptr)
-    decay_walk_kernel<true><<<dim3(n_seqs, heads, splits), dim3(threads), smem, st>>>(
-        q, q_stride, k, k_stride, qk_div, fvec, f_stride, v, v_stride, dt_dec, decay_head, skip, state, slot_stride, out,
-        seq_slot, seq_q_start, seq_q_len, heads, dim, vdim, write_state, cols_per_block, vec_qk, vec_v, vec_s, chunk);
-  else
-    decay_walk_kernel<false><<<dim3(n_seqs, heads, splits), dim3(threads), smem, st>>>(
-        q, q_stride, k, k_stride, qk_div, fvec, f_stride, v, v_stride, dt_dec, decay_head, skip, state, slot_stride, out,
-        seq_slot, seq_q_start, seq_q_len, heads, dim, vdim, write_state, cols_per_block, vec_qk, vec_v, vec_s, chunk);
+  kernel<<<dim3(n_seqs, heads, splits), dim3(threads), smem, st>>>(
+      q, q_stride, k, k_stride, qk_div, fvec, f_stride, v, v_stride, dt_dec, decay_head, skip, state, slot_stride, out,
+      seq_slot, seq_q_start, seq_q_len, heads, dim, vdim, write_state, cols_per_block, vec_qk, vec_v, vec_s, chunk, ones_out);
   return launch_status();
 }
 
@@ -393,15 +403,16 @@ TKB_EXPORT int tkb_ssm_prep(const float* proj, int stride, int xbc_off, int C, i
 
 // dt_dec: float32 [T, 2 * heads] (key scale, then decay) or null, then decay_head [heads] is the decay and the key
 // scale is 1; or fvec [T, heads * dim] (rows of f_stride floats): a decay for every key channel, key scale 1 (then
-// dt_dec and decay_head are null).  skip: [heads] or null.
+// dt_dec and decay_head are null).  skip: [heads] or null.  ones_out: float32 [T, heads] or null; given, a head's state
+// holds one more column whose value is 1 at every token, and S^T q of that column goes there (not with fvec).
 TKB_EXPORT int tkb_decay_walk(const float* q, int q_stride, const float* k, int k_stride, int qk_div, const float* fvec,
                               int f_stride, const float* v, int v_stride, const float* dt_dec, const float* decay_head, const float* skip,
                               float* state, long long slot_stride, float* out, const int* seq_slot,
                               const int* seq_q_start, const int* seq_q_len, int n_seqs, int n_tokens, int heads, int dim,
-                              int vdim, int write_state, void* st) {
-  if (fvec != nullptr && (dt_dec != nullptr || qk_div != 1)) return -2;
+                              int vdim, int write_state, float* ones_out, void* st) {
+  if (fvec != nullptr && (dt_dec != nullptr || qk_div != 1 || ones_out != nullptr)) return -2;
   return walk_launch(q, q_stride, k, k_stride, qk_div, fvec, f_stride, v, v_stride, dt_dec, decay_head, skip, state, slot_stride, out,
-                     seq_slot, seq_q_start, seq_q_len, n_seqs, n_tokens, heads, dim, vdim, write_state, (cudaStream_t)st);
+                     seq_slot, seq_q_start, seq_q_len, n_seqs, n_tokens, heads, dim, vdim, write_state, ones_out, (cudaStream_t)st);
 }
 
 TKB_EXPORT int tkb_silu_cols(float* x, int stride, int ncols, int rows, void* st) {
@@ -558,3 +569,143 @@ TKB_EXPORT int tkb_rotate_scale(float* proj, int stride, int q_off, int k_off, i
                     proj, stride, q_off, k_off, heads, dim, rot_dims, pairs, freq, positions, token_seq, q_scale,
                     k_scale);
 }
+
+namespace {
+
+// Gates of a matrix memory, one block a (request, head): with log gates i = cap tanh((zi + bi) / cap) and
+// f = log_sigmoid(cap tanh((zf + bf) / cap)) and a running maximum m_t = max(f_t + m_(t-1), i_t), the decay
+// a_t = exp(f_t + m_(t-1) - m_t), the key scale c_t = exp(i_t - m_t) and the floor exp(-m_t) of the denominator.  The
+// maximum is a scan of the pairs (f, i) under (f1, i1) then (f2, i2) = (f1 + f2, max(i1 + f2, i2)), a block's threads at
+// a time.  (The state's scale is exp(-m) whatever m is, so a rounding of m moves a, c and the floor together.)
+constexpr int GATE_THREADS = 128;
+
+__global__ void __launch_bounds__(GATE_THREADS)
+memory_gates_kernel(const float* __restrict__ z, int stride, int i_off, int f_off, const float* __restrict__ i_bias,
+                    const float* __restrict__ f_bias, float cap, float* __restrict__ state, long long slot_stride,
+                    long long m_off, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
+                    const int* __restrict__ seq_q_len, int heads, float* __restrict__ dt_dec, float* __restrict__ floor_out,
+                    int write_state) {
+  __shared__ float wf[GATE_THREADS / 32], wm[GATE_THREADS / 32];
+  __shared__ float m_last;
+  trigger_dependents();
+  const int s = blockIdx.x, h = blockIdx.y;
+  const int n = seq_q_len[s];
+  if (n <= 0) return;
+  const int start = seq_q_start[s];
+  grid_dependency_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float* mp = state + (size_t)seq_slot[s] * slot_stride + m_off + h;
+  float m0 = *mp;  // the maximum before this round of tokens
+  const float bi = i_bias[h], bf = f_bias[h], inv_cap = 1.f / cap;
+  for (int t0 = 0; t0 < n; t0 += GATE_THREADS) {
+    const int t = t0 + tid;
+    const bool live = t < n;
+    float gi = 0.f, gf = 0.f;
+    float F = 0.f, M = -INFINITY;  // past the end: the pair that changes nothing
+    if (live) {
+      const float* row = z + (size_t)(start + t) * stride;
+      gi = cap * tanhf((row[i_off + h] + bi) * inv_cap);
+      const float x = cap * tanhf((row[f_off + h] + bf) * inv_cap);
+      gf = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
+      F = gf;
+      M = gi;
+    }
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pf = __shfl_up_sync(0xffffffffu, F, o), pm = __shfl_up_sync(0xffffffffu, M, o);
+      if (lane >= o) {
+        M = fmaxf(pm + F, M);
+        F += pf;
+      }
+    }
+    if (lane == 31) {
+      wf[warp] = F;
+      wm[warp] = M;
+    }
+    __syncthreads();
+    float m_in = m0;  // the maximum before this warp's first token
+    for (int w = 0; w < warp; w++) m_in = fmaxf(m_in + wf[w], wm[w]);
+    const float m_t = fmaxf(m_in + F, M);
+    float m_prev = __shfl_up_sync(0xffffffffu, m_t, 1);
+    if (lane == 0) m_prev = m_in;
+    if (live) {
+      const size_t at = (size_t)(start + t);
+      dt_dec[at * 2 * heads + h] = expf(gi - m_t);
+      dt_dec[at * 2 * heads + heads + h] = expf(gf + (m_prev - m_t));
+      floor_out[at * heads + h] = expf(-m_t);
+    }
+    if (t == min(n, t0 + GATE_THREADS) - 1) m_last = m_t;
+    __syncthreads();
+    m0 = m_last;  // (written again only after the next round's first barrier)
+  }
+  if (write_state && tid == 0) *mp = m0;
+}
+
+// out[t][head's vdim values] = N(o) * w * sigmoid(g) * out_scale with o = S^T q / (max(|n . q|, floor) + den_eps), q scaled
+// by q_scale on the way, N the division by the head's root mean square.  raw float32 [T, heads * vdim], den and floor
+// float32 [T, heads], g float32 at column g_off of rows of g_stride.  One warp a (token, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+memory_norm_kernel(const float* __restrict__ raw, const float* __restrict__ den, const float* __restrict__ floor_in,
+                   const float* __restrict__ g, int g_stride, int g_off, const float* __restrict__ w, float q_scale,
+                   float den_eps, float eps, float out_scale, T* __restrict__ out, int out_stride, int heads, int vdim,
+                   long long pairs) {
+  trigger_dependents();
+  grid_dependency_wait();
+  const int lane = threadIdx.x & 31;
+  const long long pair = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (pair >= pairs) return;
+  const long long t = pair / heads;
+  const int h = (int)(pair - t * heads);
+  const float f = q_scale / (fmaxf(fabsf(den[pair] * q_scale), floor_in[pair]) + den_eps);
+  const float* o = raw + pair * vdim;
+  float ss = 0.f;
+  for (int j = lane; j < vdim; j += 32) {
+    const float v = o[j] * f;
+    ss = fmaf(v, v, ss);
+  }
+  ss = warp_sum(ss);
+  const float r = f * rsqrtf(ss / (float)vdim + eps) * out_scale;
+  const float* gr = g + t * g_stride + g_off + (long long)h * vdim;
+  const float* wr = w + (long long)h * vdim;
+  T* dst = out + t * out_stride + (long long)h * vdim;
+  for (int j = lane; j < vdim; j += 32) dst[j] = from_float<T>(o[j] * r * wr[j] / (1.f + expf(-gr[j])));
+}
+
+template <typename T>
+int memory_norm_launch(const float* raw, const float* den, const float* floor_in, const float* g, int g_stride, int g_off,
+                       const float* w, float q_scale, float den_eps, float eps, float out_scale, void* out, int out_stride,
+                       int heads, int vdim, int n_tokens, cudaStream_t st) {
+  if (n_tokens <= 0) return 0;
+  if (heads <= 0 || vdim <= 0 || out_stride < heads * vdim) return -2;
+  const long long pairs = (long long)n_tokens * heads;
+  const long long blocks = (pairs + 7) / 8;
+  if (blocks > 0x7fffffffLL) return -3;
+  return launch_pdl(memory_norm_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, st, raw, den, floor_in, g, g_stride, g_off, w,
+                    q_scale, den_eps, eps, out_scale, (T*)out, out_stride, heads, vdim, pairs);
+}
+
+}  // namespace
+
+TKB_EXPORT int tkb_memory_gates(const float* z, int stride, int i_off, int f_off, const float* i_bias, const float* f_bias,
+                                float cap, float* state, long long slot_stride, long long m_off, const int* seq_slot,
+                                const int* seq_q_start, const int* seq_q_len, int n_seqs, int heads, float* dt_dec,
+                                float* floor_out, int write_state, void* st) {
+  if (n_seqs <= 0) return 0;
+  if (heads <= 0 || !(cap > 0.f)) return -2;
+  if (heads > 65535) return -3;
+  return launch_pdl(memory_gates_kernel, dim3(n_seqs, heads), dim3(GATE_THREADS), 0, (cudaStream_t)st, z, stride, i_off,
+                    f_off, i_bias, f_bias, cap, state, slot_stride, m_off, seq_slot, seq_q_start, seq_q_len, heads, dt_dec,
+                    floor_out, write_state);
+}
+
+#define TKB_MEMORY_NORM_EXPORT(SUF, T)                                                                                \
+  TKB_EXPORT int tkb_memory_norm_##SUF(const float* raw, const float* den, const float* floor_in, const float* g,     \
+                                       int g_stride, int g_off, const float* w, float q_scale, float den_eps,         \
+                                       float eps, float out_scale, void* out, int out_stride, int heads, int vdim,    \
+                                       int n_tokens, void* st) {                                                      \
+    return memory_norm_launch<T>(raw, den, floor_in, g, g_stride, g_off, w, q_scale, den_eps, eps, out_scale, out,    \
+                                 out_stride, heads, vdim, n_tokens, (cudaStream_t)st);                                \
+  }
+TKB_MEMORY_NORM_EXPORT(f32, float)
+TKB_MEMORY_NORM_EXPORT(bf16, __nv_bfloat16)

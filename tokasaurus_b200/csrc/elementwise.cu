@@ -77,14 +77,32 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = u;
 }
 
-// MODE: 0 no update, 1 update in the activation type, 2 update as float32 slices.  One instantiation a mode,
+// The update as float32 slices: n of them, spaced `stride` floats apart; SECOND: followed by the n2 slices of a second
+// update (a block whose two sublayers read one norm leaves two), counted on.
+struct Slices {
+  const float* p;
+  int n;
+  long long stride;
+  const float* p2;
+  int n2;
+  long long stride2;
+};
+template <bool SECOND> __device__ __forceinline__ int slice_count(const Slices& s) { return SECOND ? s.n + s.n2 : s.n; }
+template <bool SECOND> __device__ __forceinline__ const float* slice_at(const Slices& s, int i) {
+  if (SECOND && i >= s.n) return s.p2 + (size_t)(i - s.n) * s.stride2;
+  return s.p + (size_t)i * s.stride;
+}
+
+// MODE: 0 no update, 1 update in the activation type, 2 update as float32 slices, 3 two such updates.  One
+// instantiation a mode,
 // and only two steps' worth of values kept in registers: with many rows (a prompt) what matters is how many
 // rows an SM holds at once, and that is set by the registers a thread takes.
 template <typename T, int MODE, int MAXT>
 __global__ void __launch_bounds__(MAXT, MAXT <= 256 ? 6 : 2)
-add_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ partials,
-                   int n_partials, long long partial_stride, const float* __restrict__ w, T* __restrict__ out,
-                   float eps, int H) {
+add_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, Slices sl, const float* __restrict__ w,
+                   T* __restrict__ out, float eps, int H) {
+  constexpr bool SECOND = MODE == 3;
+  const int n_partials = MODE >= 2 ? slice_count<SECOND>(sl) : 0;
   trigger_dependents();
   __shared__ float scratch[33];
   const size_t base = (size_t)blockIdx.x * H;
@@ -106,15 +124,15 @@ add_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, const flo
     // x + update of four elements at 4 * i4, stored back
     auto updated = [&](int i4) {
       float4 v = load4(xr + 4 * i4);
-      if (MODE == 2) {
+      if (MODE >= 2) {
         // float32 slices of a split matrix product: four loads in flight together, added in slice order
         float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
-        const float* src = partials + base + 4 * i4;
+        const size_t at = base + 4 * i4;
         for (int p0 = 0; p0 < n_partials; p0 += 4) {
           float4 q[4];
 #pragma unroll
           for (int j = 0; j < 4; j++)
-            q[j] = p0 + j < n_partials ? load4(src + (size_t)(p0 + j) * partial_stride) : make_float4(0.f, 0.f, 0.f, 0.f);
+            q[j] = p0 + j < n_partials ? load4(slice_at<SECOND>(sl, p0 + j) + at) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
           for (int j = 0; j < 4; j++) {
             if (p0 + j < n_partials) {
@@ -155,10 +173,10 @@ add_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, const flo
     return;
   }
   grid_dependency_wait();
-  if (MODE == 2) {
+  if (MODE >= 2) {
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
       float d = 0.f;
-      for (int p = 0; p < n_partials; p++) d += partials[(size_t)p * partial_stride + base + i];
+      for (int p = 0; p < n_partials; p++) d += slice_at<SECOND>(sl, p)[base + i];
       float v = xr[i] + d;
       xr[i] = v;
       ss += v * v;
@@ -188,10 +206,10 @@ add_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, const flo
 // from global memory instead, so the result does not depend on the wait.
 __device__ __forceinline__ uint32_t ew_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
-template <typename T>
-__global__ void add_rmsnorm_bulk_kernel(float* __restrict__ x, const float* __restrict__ partials, int n_partials,
-                                        long long partial_stride, const float* __restrict__ w, T* __restrict__ out,
+template <typename T, bool SECOND>
+__global__ void add_rmsnorm_bulk_kernel(float* __restrict__ x, Slices sl, const float* __restrict__ w, T* __restrict__ out,
                                         float eps, int H) {
+  const int n_partials = slice_count<SECOND>(sl);
   extern __shared__ __align__(128) unsigned char ew_smem[];
   float* rows = reinterpret_cast<float*>(ew_smem);  // [1 + n_partials][H]
   __shared__ __align__(8) unsigned long long bar;
@@ -222,7 +240,7 @@ __global__ void add_rmsnorm_bulk_kernel(float* __restrict__ x, const float* __re
                  ::"r"(ew_smem_u32(rows)), "l"(xr), "r"(row_bytes), "r"(bar_a) : "memory");
     for (int p = 0; p < n_partials; p++)
       asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                   ::"r"(ew_smem_u32(rows + (size_t)(p + 1) * H)), "l"(partials + (size_t)p * partial_stride + base),
+                   ::"r"(ew_smem_u32(rows + (size_t)(p + 1) * H)), "l"(slice_at<SECOND>(sl, p) + base),
                      "r"(row_bytes), "r"(bar_a) : "memory");
   }
   bool arrived = false;
@@ -244,7 +262,7 @@ __global__ void add_rmsnorm_bulk_kernel(float* __restrict__ x, const float* __re
     } else {
       v = load4(xr + 4 * i4);
       for (int p = 0; p < n_partials; p++) {
-        const float4 q = load4(partials + (size_t)p * partial_stride + base + 4 * i4);
+        const float4 q = load4(slice_at<SECOND>(sl, p) + base + 4 * i4);
         d.x += q.x; d.y += q.y; d.z += q.z; d.w += q.w;
       }
     }
@@ -275,55 +293,64 @@ __global__ void add_rmsnorm_bulk_kernel(float* __restrict__ x, const float* __re
   }
 }
 
+template <typename T, bool SECOND>
+static int add_rmsnorm_bulk_launch(float* x, Slices sl, size_t bulk_bytes, const float* w, void* out, float eps, int rows,
+                                   int H, cudaStream_t st) {
+  static bool attr_done = false;
+  if (!attr_done) {
+    cudaError_t e = cudaFuncSetAttribute(add_rmsnorm_bulk_kernel<T, SECOND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    attr_done = true;
+  }
+  return launch_pdl(add_rmsnorm_bulk_kernel<T, SECOND>, dim3(rows), dim3(H >= 2048 ? 512 : 256), bulk_bytes, st, x, sl, w,
+                    (T*)out, eps, H);
+}
+
 template <typename T>
-static int add_rmsnorm_launch(float* x, const void* delta, const float* partials, int n_partials,
-                              long long partial_stride, const float* w, void* out, float eps, int rows, int H,
+static int add_rmsnorm_launch(float* x, const void* delta, Slices sl, const float* w, void* out, float eps, int rows, int H,
                               cudaStream_t st) {
   if (rows <= 0) return 0;
+  if ((sl.p == nullptr && sl.p2 != nullptr) || (sl.p != nullptr && (sl.n < 1 || (sl.p2 != nullptr && sl.n2 < 1)))) return -2;
   // few rows with slices: bulk copies into shared memory (rows of 16-byte multiples, everything 16-byte aligned)
-  const size_t bulk_bytes = (size_t)(n_partials + 1) * H * 4;
-  if (partials != nullptr && rows <= 64 && (H & 3) == 0 && bulk_bytes <= 200 * 1024 && ((uintptr_t)x & 15) == 0 &&
-      ((uintptr_t)partials & 15) == 0 && (partial_stride & 3) == 0) {
-    static bool attr_done[2] = {false, false};
-    constexpr int which = sizeof(T) == 4 ? 0 : 1;
-    if (!attr_done[which]) {
-      cudaError_t e = cudaFuncSetAttribute(add_rmsnorm_bulk_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-      if (e != cudaSuccess) return (int)e;
-      attr_done[which] = true;
-    }
-    return launch_pdl(add_rmsnorm_bulk_kernel<T>, dim3(rows), dim3(H >= 2048 ? 512 : 256), bulk_bytes, st, x, partials,
-                      n_partials, partial_stride, w, (T*)out, eps, H);
+  const size_t bulk_bytes = (size_t)(1 + sl.n + (sl.p2 != nullptr ? sl.n2 : 0)) * H * 4;
+  if (sl.p != nullptr && rows <= 64 && (H & 3) == 0 && bulk_bytes <= 200 * 1024 && ((uintptr_t)x & 15) == 0 &&
+      ((uintptr_t)sl.p & 15) == 0 && (sl.stride & 3) == 0 && ((uintptr_t)sl.p2 & 15) == 0 && (sl.stride2 & 3) == 0) {
+    return sl.p2 != nullptr ? add_rmsnorm_bulk_launch<T, true>(x, sl, bulk_bytes, w, out, eps, rows, H, st)
+                            : add_rmsnorm_bulk_launch<T, false>(x, sl, bulk_bytes, w, out, eps, rows, H, st);
   }
   // few rows: many threads a row, they hide the latency; many rows: several rows an SM in flight do
   int threads = H >= 8192 || (H >= 2048 && rows < 592) ? 512 : (H >= 512 ? 256 : 128);
 #define TKB_NORM(MODE, MAXT)                                                                                        \
-  return launch_pdl(add_rmsnorm_kernel<T, MODE, MAXT>, dim3(rows), dim3(threads), 0, st, x, (const T*)delta, partials, \
-                    n_partials, partial_stride, w, (T*)out, eps, H)
-  const int mode = partials != nullptr ? 2 : (delta != nullptr ? 1 : 0);
+  return launch_pdl(add_rmsnorm_kernel<T, MODE, MAXT>, dim3(rows), dim3(threads), 0, st, x, (const T*)delta, sl, w, \
+                    (T*)out, eps, H)
+  const int mode = sl.p2 != nullptr ? 3 : (sl.p != nullptr ? 2 : (delta != nullptr ? 1 : 0));
   if (threads <= 256) {  // up to 256 threads a row: six rows an SM (40 registers a thread)
+    if (mode == 3) TKB_NORM(3, 256);
     if (mode == 2) TKB_NORM(2, 256);
     if (mode == 1) TKB_NORM(1, 256);
     TKB_NORM(0, 256);
   }
+  if (mode == 3) TKB_NORM(3, 512);
   if (mode == 2) TKB_NORM(2, 512);
   if (mode == 1) TKB_NORM(1, 512);
   TKB_NORM(0, 512);
 #undef TKB_NORM
 }
 // delta: update in the activation type [rows, H], or null.  partials: the update as float32 slices
-// [n_partials][rows, H] spaced partial_stride floats apart, or null.  At most one of the two.
-TKB_EXPORT int tkb_add_rmsnorm_f32(float* x, const void* delta, const float* partials, int n_partials,
-                                   long long partial_stride, const float* w, void* out, float eps, int rows, int H,
-                                   void* st) {
-  return add_rmsnorm_launch<float>(x, delta, partials, n_partials, partial_stride, w, out, eps, rows, H,
-                                   (cudaStream_t)st);
-}
-TKB_EXPORT int tkb_add_rmsnorm_bf16(float* x, const void* delta, const float* partials, int n_partials,
-                                    long long partial_stride, const float* w, void* out, float eps, int rows, int H,
-                                    void* st) {
-  return add_rmsnorm_launch<__nv_bfloat16>(x, delta, partials, n_partials, partial_stride, w, out, eps, rows, H,
-                                           (cudaStream_t)st);
-}
+// [n_partials][rows, H] spaced partial_stride floats apart, or null.  At most one of the two.  partials2 (with
+// partials; or null): the slices of a second update, added behind the first's.
+#define TKB_ADD_RMSNORM_EXPORT(SUF, T)                                                                              \
+  TKB_EXPORT int tkb_add_rmsnorm_##SUF(float* x, const void* delta, const float* partials, int n_partials,          \
+                                       long long partial_stride, const float* partials2, int n_partials2,           \
+                                       long long partial_stride2, const float* w, void* out, float eps, int rows,   \
+                                       int H, void* st) {                                                           \
+    return add_rmsnorm_launch<T>(x, delta,                                                                          \
+                                 Slices{partials, n_partials, partial_stride, partials2, n_partials2,               \
+                                        partial_stride2},                                                           \
+                                 w, out, eps, rows, H, (cudaStream_t)st);                                           \
+  }
+TKB_ADD_RMSNORM_EXPORT(f32, float)
+TKB_ADD_RMSNORM_EXPORT(bf16, __nv_bfloat16)
 
 // ------------------------------------------------------------------------------------------------
 // From a step's q|k|v rows to rotated q and to the cache: rotary position encoding of q and k (half-split
@@ -797,6 +824,64 @@ TKB_EXPORT int tkb_gelu_tanh_mul_f32(const void* gu, void* out, int rows, int I,
 }
 TKB_EXPORT int tkb_gelu_tanh_mul_bf16(const void* gu, void* out, int rows, int I, int interleave, void* st) {
   return silu_mul_launch<__nv_bfloat16, 1>(gu, out, rows, I, interleave, (cudaStream_t)st);
+}
+
+// ------------------------------------------------------------------------------------------------
+// out = gelu(z), the exact (erf) form, for an up product without a gate.  z: float32 slices of a K-split product
+// ([n_slices][total], added in slice order), or values in the activation type (z_act).  Four elements a thread where
+// the count allows.
+__device__ __forceinline__ float gelu_erf_f(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
+template <typename T>
+__global__ void gelu_rows_kernel(const float* __restrict__ z, int n_slices, long long stride, const T* __restrict__ z_act,
+                                 T* __restrict__ out, long long total) {
+  trigger_dependents();
+  grid_dependency_wait();
+  const long long step = (long long)gridDim.x * blockDim.x;
+  if ((total & 3) == 0 && (stride & 3) == 0) {
+    for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < total; i += step * 4) {
+      float4 v;
+      if (z_act != nullptr) {
+        v = load4(z_act + i);
+      } else {
+        v = load4(z + i);
+        for (int s = 1; s < n_slices; s++) {
+          const float4 q = load4(z + (size_t)s * stride + i);
+          v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
+        }
+      }
+      store4(out + i, make_float4(gelu_erf_f(v.x), gelu_erf_f(v.y), gelu_erf_f(v.z), gelu_erf_f(v.w)));
+    }
+    return;
+  }
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += step) {
+    float v;
+    if (z_act != nullptr) {
+      v = to_float(z_act[i]);
+    } else {
+      v = z[i];
+      for (int s = 1; s < n_slices; s++) v += z[(size_t)s * stride + i];
+    }
+    out[i] = from_float<T>(gelu_erf_f(v));
+  }
+}
+template <typename T>
+static int gelu_rows_launch(const float* z, int n_slices, long long stride, const void* z_act, void* out, long long total,
+                            cudaStream_t st) {
+  if (total <= 0) return 0;
+  if ((z == nullptr) == (z_act == nullptr) || (z != nullptr && n_slices < 1)) return -2;
+  long long blocks = (total / 4 + 255) / 256;
+  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+  if (blocks < 1) blocks = 1;
+  return launch_pdl(gelu_rows_kernel<T>, dim3((int)blocks), dim3(256), 0, st, z, n_slices, stride, (const T*)z_act, (T*)out,
+                    total);
+}
+TKB_EXPORT int tkb_gelu_rows_f32(const float* z, int n_slices, long long stride, const void* z_act, void* out,
+                                 long long total, void* st) {
+  return gelu_rows_launch<float>(z, n_slices, stride, z_act, out, total, (cudaStream_t)st);
+}
+TKB_EXPORT int tkb_gelu_rows_bf16(const float* z, int n_slices, long long stride, const void* z_act, void* out,
+                                  long long total, void* st) {
+  return gelu_rows_launch<__nv_bfloat16>(z, n_slices, stride, z_act, out, total, (cudaStream_t)st);
 }
 
 // ------------------------------------------------------------------------------------------------

@@ -43,7 +43,7 @@ __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     bf16* __restrict__ out, int ldo, int M, int N, int K, int* __restrict__ status,
                     const int* __restrict__ tile_group, int group_rows, float act_limit, float act_alpha,
-                    int plain_act) {
+                    int plain_act, const float* __restrict__ row_scale) {
   extern __shared__ unsigned char smem_raw[];
   constexpr int STAGES = Cfg<BN>::STAGES;
   __shared__ __align__(8) uint64_t full_bar[STAGES], empty_bar[STAGES], acc_full[2], acc_empty[2];
@@ -143,6 +143,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       if (!mbar_wait(&acc_full[buf], (j >> 1) & 1)) { failed = 1; ok = false; break; }
       tcgen05_fence_after();
       const int row = m0 + q * 32 + lane;
+      // a factor on a whole row of A is a factor on the row of the accumulator
+      const float rs = GATED && row_scale != nullptr && row < M ? row_scale[row] : 1.f;
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += 32) {
         uint32_t r[32];
@@ -174,6 +176,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             }
           } else {
             // columns come in groups of 16: 8 gate columns, then the 8 up columns of the same features
+            if (row_scale != nullptr) {
+#pragma unroll
+              for (int jj = 0; jj < 32; jj++) r[jj] = __float_as_uint(__uint_as_float(r[jj]) * rs);
+            }
 #pragma unroll
             for (int g = 0; g < 2; g++) {
               const int n = n0 + c0 + 16 * g;
@@ -220,7 +226,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 template <int BN, bool GATED>
 int launch(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M, int N, int K, int* status,
            cudaStream_t st, const int* tile_group = nullptr, int groups = 1, float act_limit = 0.f,
-           float act_alpha = 0.f, int plain_act = 0) {
+           float act_alpha = 0.f, int plain_act = 0, const float* row_scale = nullptr) {
   static bool attr_done = false;
   if (!attr_done) {
     cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -237,17 +243,19 @@ int launch(const void* A, int lda, const void* W, int ldw, void* out, int ldo, i
   const int tiles = ((N + BN - 1) / BN) * ((M + BM - 1) / BM);
   dim3 grid(tiles < n_sms ? tiles : n_sms);
   gemm_tcgen05_kernel<BN, GATED><<<grid, THREADS, Cfg<BN>::SMEM_BYTES, st>>>(map_a, map_w, (bf16*)out, ldo, M, N, K, status,
-                                                                                 tile_group, N, act_limit, act_alpha, plain_act);
+                                                                                 tile_group, N, act_limit, act_alpha, plain_act, row_scale);
   return launch_status();
 }
 
 }  // namespace
 
-// out[M, N] (bfloat16, row stride ldo) = A[M, K] . W[N, K]^T.  gated != 0: W interleaves gate/up rows in groups of
-// 8 and out is [M, N/2] = silu(gate) * up.  K and the row strides must be multiples of 8 elements and the base
+// out[M, N] (bfloat16, row stride ldo) = A[M, K] . W[N, K]^T.  gated == 1: W interleaves gate/up rows in groups of
+// 8 and out is [M, N/2] = silu(gate) * up; gated == 2: ungated, the exact GELU of every result.  K and the row strides must be multiples of 8 elements and the base
 // addresses 16-byte aligned (what a TMA descriptor asks for); N a multiple of 16 for the gated form.
 TKB_EXPORT int tkb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M, int N,
                                      int K, int gated, int* status, void* st_) {
+  const int plain_act = gated == 2 ? 1 : 0;
+  if (gated == 2) gated = 0;
   cudaStream_t st = (cudaStream_t)st_;
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (lda & 7) || (ldw & 7) || (((uintptr_t)A) & 15) || (((uintptr_t)W) & 15)) return -2;
@@ -256,10 +264,10 @@ TKB_EXPORT int tkb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int 
   if (rc) return rc;
   if (N >= 256) {
     return gated ? launch<256, true>(A, lda, W, ldw, out, ldo, M, N, K, status, st)
-                 : launch<256, false>(A, lda, W, ldw, out, ldo, M, N, K, status, st);
+                 : launch<256, false>(A, lda, W, ldw, out, ldo, M, N, K, status, st, nullptr, 1, 0.f, 0.f, plain_act);
   }
   return gated ? launch<128, true>(A, lda, W, ldw, out, ldo, M, N, K, status, st)
-               : launch<128, false>(A, lda, W, ldw, out, ldo, M, N, K, status, st);
+               : launch<128, false>(A, lda, W, ldw, out, ldo, M, N, K, status, st, nullptr, 1, 0.f, 0.f, plain_act);
 }
 
 // The gated form with another activation in its epilogue: g = min(gate, limit), u = clamp(up, -limit, limit),
@@ -280,22 +288,23 @@ TKB_EXPORT int tkb_gemm_tcgen05_clamped_bf16(const void* A, int lda, const void*
 // rows) multiplies the weights of group tile_group[i] (a device array of ceil(M / 128) entries; -1: the tile is
 // nobody's and is left out).  The caller orders A's rows by group and starts every group on a tile boundary.
 // gated: 0 plain, 1 silu(gate) * up over interleaved rows, 2 plain with the exact GELU of every result.
+// row_scale (gated == 1; float32 [M] or null): row i of A counts row_scale[i] times, applied to the accumulator.
 TKB_EXPORT int tkb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M,
-                                             int N, int K, int gated, const int* tile_group, int groups, int* status,
-                                             void* st_) {
+                                             int N, int K, int gated, const int* tile_group, int groups,
+                                             const float* row_scale, int* status, void* st_) {
   const int plain_act = gated == 2 ? 1 : 0;
   if (gated == 2) gated = 0;
   cudaStream_t st = (cudaStream_t)st_;
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (lda & 7) || (ldw & 7) || (((uintptr_t)A) & 15) || (((uintptr_t)W) & 15)) return -2;
-  if (groups <= 0 || tile_group == nullptr || (gated && (N & 15))) return -2;
+  if (groups <= 0 || tile_group == nullptr || (gated && (N & 15)) || (row_scale != nullptr && !gated)) return -2;
   int rc = get_encode();
   if (rc) return rc;
   if (N >= 256) {
-    return gated ? launch<256, true>(A, lda, W, ldw, out, ldo, M, N, K, status, st, tile_group, groups)
+    return gated ? launch<256, true>(A, lda, W, ldw, out, ldo, M, N, K, status, st, tile_group, groups, 0.f, 0.f, 0, row_scale)
                  : launch<256, false>(A, lda, W, ldw, out, ldo, M, N, K, status, st, tile_group, groups, 0.f, 0.f, plain_act);
   }
-  return gated ? launch<128, true>(A, lda, W, ldw, out, ldo, M, N, K, status, st, tile_group, groups)
+  return gated ? launch<128, true>(A, lda, W, ldw, out, ldo, M, N, K, status, st, tile_group, groups, 0.f, 0.f, 0, row_scale)
                : launch<128, false>(A, lda, W, ldw, out, ldo, M, N, K, status, st, tile_group, groups, 0.f, 0.f, plain_act);
 }
 

@@ -6,7 +6,11 @@
 // A second way of choosing (moe_choose_scored): scores s = sigmoid(logits); the choice goes by s + correction (a
 // learned vector that takes no part in the weights), among the experts of the best `keep` of `groups` equal groups of
 // neighbours only (a group scores the sum of its two largest choice scores); the weights are the chosen experts' s over
-// their sum (+ 1e-20), times a scale.  A second kind of expert: down(gelu(up h)) with the exact (erf) GELU, no gate.
+// their sum (+ 1e-20), times a scale, or (renorm == 0) s times a scale as it is.  A second kind of expert:
+// down(gelu(up h)) with the exact (erf) GELU, no gate.
+// Weights on the way IN: with pair_scale (float32, one number a (token, choice) pair) an expert reads w * h instead of h,
+// and the outputs are added up unweighed.  A factor on a row of the operand is a factor on the row of the product, so
+// the first product's sums are multiplied before the activation sees them.
 #include "common.cuh"
 #include <float.h>
 
@@ -142,11 +146,11 @@ moe_choose_kernel(const float* __restrict__ z_all, const int* __restrict__ token
 // Router, second kernel, the other way of choosing: one warp a token.  s = sigmoid(z), c = s + correction; group g holds
 // experts g * per .. (g + 1) * per - 1 and scores the sum of its two largest c (its only c if per == 1); experts
 // outside the `keep` best groups cannot be chosen (their c counts as minus infinity); the `top` largest c are chosen,
-// equal scores: the lower expert (group) first; weights s / (sum of the chosen s + 1e-20) * scale.
+// equal scores: the lower expert (group) first; weights s / (sum of the chosen s + 1e-20) * scale, or s * scale (renorm 0).
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_choose_scored_kernel(const float* __restrict__ z_all, const float* __restrict__ correction,
                          const int* __restrict__ token_seq, int* __restrict__ top_idx, float* __restrict__ top_w,
-                         int n_tokens, int E, int top, int groups, int keep, float scale) {
+                         int n_tokens, int E, int top, int groups, int keep, float scale, int renorm) {
   extern __shared__ float zs[];  // [warps][2 E + groups]: s, c, group scores
   trigger_dependents();
   grid_dependency_wait();
@@ -224,7 +228,7 @@ moe_choose_scored_kernel(const float* __restrict__ z_all, const float* __restric
     }
     __syncwarp();
   }
-  const float f = scale / (denom + 1e-20f);
+  const float f = renorm ? scale / (denom + 1e-20f) : scale;
   for (int k = lane; k < top; k += 32) top_w[(size_t)t * top + k] *= f;
 }
 
@@ -283,14 +287,17 @@ __global__ void moe_order_kernel(const int* __restrict__ top_idx, int n_pairs, i
   }
 }
 
-// dst[p] = src[src_token[p]] (zeros where src_token[p] < 0): the step's rows in the order of the experts' spans.
+// dst[p] = src[src_token[p]] (zeros where src_token[p] < 0): the step's rows in the order of the experts' spans; and, if
+// asked, place_scale[p] = pair_scale[order[p]] (0 at the padding, where order holds nothing).
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ src, const int* __restrict__ src_token, T* __restrict__ dst,
-                                  int H) {
+                                  int H, const int* __restrict__ order, const float* __restrict__ pair_scale,
+                                  float* __restrict__ place_scale) {
   trigger_dependents();
   grid_dependency_wait();
   const int p = blockIdx.x;
   const int t = src_token[p];
+  if (place_scale != nullptr && threadIdx.x == 0) place_scale[p] = t >= 0 ? pair_scale[order[p]] : 0.f;
   T* d = dst + (size_t)p * H;
   if (t < 0) {
     for (int i = threadIdx.x; i < H; i += blockDim.x) d[i] = from_float<T>(0.f);
@@ -321,7 +328,7 @@ template <typename TA, typename TC, int ACT>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC* __restrict__ C, int ldc,
                 const int* __restrict__ offsets, const int* __restrict__ order, int top, int E, int N, int K,
-                float limit, float alpha) {
+                float limit, float alpha, const float* __restrict__ pair_scale) {
   constexpr bool GATED = ACT == ACT_GATED || ACT == ACT_CLAMPED;
   __shared__ float As[BK][BM + 4];
   __shared__ float Ws[BK][BN + 4];
@@ -394,11 +401,16 @@ moe_gemm_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC*
   for (int i = 0; i < 4; i++) {
     const int p = p0 + ty * 4 + i;
     if (p >= p1) continue;
+    const float ps = ACT == ACT_GATED && pair_scale != nullptr ? pair_scale[order[p]] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       float v = acc[i][j];
+      if (ACT == ACT_GATED && pair_scale != nullptr) {
+        v *= ps;
+        acu[GATED ? i : 0][j] *= ps;
+      }
       if (ACT == ACT_CLAMPED) v = clamped_unit(v, acu[i][j], limit, alpha);
       else if (GATED) v = v / (1.f + expf(-v)) * acu[i][j];
       if (ACT == ACT_GELU) v = gelu_erf_f(v);
@@ -440,7 +452,7 @@ template <typename TA, typename TC, int ACT>
 __global__ void __launch_bounds__(GV_WARPS * 32)
 moe_gemv_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC* __restrict__ C, int ldc,
                 const int* __restrict__ offsets, const int* __restrict__ order, int top, int N, int K, float limit,
-                float alpha) {
+                float alpha, const float* __restrict__ pair_scale) {
   constexpr bool GATED = ACT == ACT_GATED || ACT == ACT_CLAMPED;
   trigger_dependents();
   grid_dependency_wait();
@@ -496,11 +508,16 @@ moe_gemv_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC*
 #pragma unroll
       for (int r = 0; r < GV_ROWS; r++) {
         if (r < nr) {
+          const float ps = ACT == ACT_GATED && pair_scale != nullptr ? pair_scale[order[r0 + r]] : 1.f;
 #pragma unroll
           for (int j = 0; j < 2; j++) {
             float v = warp_sum(acc[j][r]);
             if (GATED) {
-              const float u = warp_sum(acu[j][r]);
+              float u = warp_sum(acu[j][r]);
+              if (ACT == ACT_GATED && pair_scale != nullptr) {
+                v *= ps;
+                u *= ps;
+              }
               v = ACT == ACT_CLAMPED ? clamped_unit(v, u, limit, alpha) : v / (1.f + expf(-v)) * u;
             }
             if (ACT == ACT_GELU) v = gelu_erf_f(v);
@@ -513,7 +530,8 @@ moe_gemv_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC*
   }
 }
 
-// out[t] = sum_k top_w[t, k] * y[place_of[t * top + k]]  (+ shared[t]), in choice order, float32 sums, rounded once.
+// out[t] = sum_k top_w[t, k] * y[place_of[t * top + k]]  (+ shared[t]), in choice order, float32 sums, rounded once
+// (top_w null: the outputs count once each).
 // shared: [rows, H] in the activation type, or float32 slices [n_slices][rows, H] added in slice order; shared_gate
 // (float32 [rows], or null): the shared part is multiplied by sigmoid(shared_gate[t]) before it is added.
 template <typename T, typename TY>
@@ -529,7 +547,7 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
     float acc = 0.f;
     for (int k = 0; k < top; k++) {
       const int p = place_of[(size_t)t * top + k];
-      if (p >= 0) acc = fmaf(top_w[(size_t)t * top + k], to_float(y[(size_t)p * H + i]), acc);
+      if (p >= 0) acc = fmaf(top_w ? top_w[(size_t)t * top + k] : 1.f, to_float(y[(size_t)p * H + i]), acc);
     }
     if (shared_gate == nullptr) {
       if (shared_t != nullptr) acc += to_float(shared_t[(size_t)t * H + i]);
@@ -559,7 +577,7 @@ int route_launch(const void* h, const float* wr, const float* br, const int* tok
 template <typename T>
 int route_scored_launch(const void* h, const float* wr, const float* br, const float* correction, const int* token_seq,
                         int* top_idx, float* top_w, float* logits, int n_tokens, int H, int E, int top, int groups,
-                        int keep, float scale, cudaStream_t st) {
+                        int keep, float scale, int renorm, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
       top > keep * (E / groups) || (size_t)(2 * E + groups) * 4 * ROUTE_WARPS > 48 * 1024 || (E + 3) / 4 > 65535)
@@ -570,23 +588,25 @@ int route_scored_launch(const void* h, const float* wr, const float* br, const f
   if (rc != 0) return rc;
   return launch_pdl(moe_choose_scored_kernel, dim3(tb), dim3(ROUTE_WARPS * 32),
                     (size_t)ROUTE_WARPS * (2 * E + groups) * sizeof(float), st, (const float*)logits, correction,
-                    token_seq, top_idx, top_w, n_tokens, E, top, groups, keep, scale);
+                    token_seq, top_idx, top_w, n_tokens, E, top, groups, keep, scale, renorm);
 }
 
 template <typename TA, typename TC, int ACT>
 int gemm_launch(const void* A, int lda, const void* W, void* C, int ldc, const int* offsets, const int* order, int top,
-                int n_places, int E, int N, int K, cudaStream_t st, float limit = 0.f, float alpha = 0.f) {
+                int n_places, int E, int N, int K, cudaStream_t st, float limit = 0.f, float alpha = 0.f,
+                const float* pair_scale = nullptr) {
   if (n_places <= 0 || N <= 0) return 0;
-  if (K <= 0 || E <= 0) return -2;
+  if (K <= 0 || E <= 0 || (pair_scale != nullptr && order == nullptr)) return -2;
   // few rows: every weight once, at full width (rows of 8 values must start on 16 bytes)
   const bool wide = K % 8 == 0 && lda % 8 == 0 && (((uintptr_t)A) & 15) == 0 && (((uintptr_t)W) & 15) == 0;
   if (wide && n_places <= GEMV_PLACES_MAX && E <= 65535)
     return launch_pdl(moe_gemv_kernel<TA, TC, ACT>, dim3((N + GV_FEATS - 1) / GV_FEATS, E), dim3(GV_WARPS * 32), 0, st,
-                      (const TA*)A, lda, (const TA*)W, (TC*)C, ldc, offsets, order, top, N, K, limit, alpha);
+                      (const TA*)A, lda, (const TA*)W, (TC*)C, ldc, offsets, order, top, N, K, limit, alpha,
+                      pair_scale);
   const int row_tiles = n_places / BM + E;  // sum over experts of ceil(count / BM) is at most this
   if (row_tiles > 65535) return -3;
   return launch_pdl(moe_gemm_kernel<TA, TC, ACT>, dim3((N + BN - 1) / BN, row_tiles), dim3(256), 0, st, (const TA*)A,
-                    lda, (const TA*)W, (TC*)C, ldc, offsets, order, top, E, N, K, limit, alpha);
+                    lda, (const TA*)W, (TC*)C, ldc, offsets, order, top, E, N, K, limit, alpha, pair_scale);
 }
 
 template <typename T, typename TY>
@@ -623,8 +643,10 @@ TKB_EXPORT int tkb_moe_order(const int* top_idx, int n_pairs, int E, int top, in
                       dim3(ROUTE_WARPS * 32), 0, (cudaStream_t)st, (const T*)h, wr, br, logits, n_tokens, H, E);       \
   }                                                                                                                    \
   TKB_EXPORT int tkb_moe_gemm_gated_##SUF(const void* A, int lda, const void* W, void* C, int ldc, const int* offsets, \
-                                          const int* order, int top, int n_places, int E, int N, int K, void* st) {    \
-    return gemm_launch<T, T, ACT_GATED>(A, lda, W, C, ldc, offsets, order, top, n_places, E, N, K, (cudaStream_t)st);  \
+                                          const int* order, int top, int n_places, int E, int N, int K,                \
+                                          const float* pair_scale, void* st) {                                         \
+    return gemm_launch<T, T, ACT_GATED>(A, lda, W, C, ldc, offsets, order, top, n_places, E, N, K, (cudaStream_t)st,   \
+                                        0.f, 0.f, pair_scale);                                                         \
   }                                                                                                                    \
   TKB_EXPORT int tkb_moe_gemm_clamped_##SUF(const void* A, int lda, const void* W, void* C, int ldc,                   \
                                             const int* offsets, const int* order, int top, int n_places, int E, int N, \
@@ -640,9 +662,9 @@ TKB_EXPORT int tkb_moe_order(const int* top_idx, int n_pairs, int E, int top, in
   TKB_EXPORT int tkb_moe_route_scored_##SUF(const void* h, const float* wr, const float* br, const float* correction,  \
                                             const int* token_seq, int* top_idx, float* top_w, float* logits,           \
                                             int n_tokens, int H, int E, int top, int groups, int keep, float scale,    \
-                                            void* st) {                                                                \
+                                            int renorm, void* st) {                                                                \
     return route_scored_launch<T>(h, wr, br, correction, token_seq, top_idx, top_w, logits, n_tokens, H, E, top,       \
-                                  groups, keep, scale, (cudaStream_t)st);                                              \
+                                  groups, keep, scale, renorm, (cudaStream_t)st);                                              \
   }                                                                                                                    \
   TKB_EXPORT int tkb_moe_gemm_##SUF(const void* A, int lda, const void* W, void* C, int ldc, const int* offsets,       \
                                     const int* order, int top, int n_places, int E, int N, int K, void* st) {          \
@@ -656,10 +678,11 @@ TKB_EXPORT int tkb_moe_order(const int* top_idx, int n_pairs, int E, int top, in
                                     H, top, shared_gate, (cudaStream_t)st);                                            \
   }                                                                                                                    \
   TKB_EXPORT int tkb_moe_gather_##SUF(const void* src, const int* src_token, void* dst, int n_places, int H,           \
-                                      void* st) {                                                                      \
+                                      const int* order, const float* pair_scale, float* place_scale, void* st) {       \
     if (n_places <= 0) return 0;                                                                                       \
+    if (place_scale != nullptr && (order == nullptr || pair_scale == nullptr)) return -2;                              \
     return launch_pdl(moe_gather_kernel<T>, dim3(n_places), dim3(H >= 1024 ? 256 : 128), 0, (cudaStream_t)st,          \
-                      (const T*)src, src_token, (T*)dst, H);                                                           \
+                      (const T*)src, src_token, (T*)dst, H, order, pair_scale, place_scale);                           \
   }
 
 TKB_MOE_EXPORTS(f32, float)

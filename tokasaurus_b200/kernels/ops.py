@@ -135,27 +135,38 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, token_seq: torch.Tensor
              c_int(H), c_int(V), c_float(scale), _ptr(status), _stream()), "embed_gather")
 
 
-def add_rmsnorm(x: torch.Tensor, delta: torch.Tensor | None, weight: torch.Tensor, eps: float,
-                out: torch.Tensor) -> None:
+def add_rmsnorm(x: torch.Tensor, delta, weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
     """x += delta (float32, in place) if delta is given; out = rmsnorm(x) * weight in out's dtype.
 
-    ``delta`` is [rows, H] in out's dtype, or float32 [slices, rows, H]: the slices of a split matrix
-    product (``linear_smallm``), added in slice order."""
-    _need_cuda(x, delta, weight, out)
+    ``delta`` is [rows, H] in out's dtype or float32, or float32 [slices, rows, H]: the slices of a split matrix
+    product (``linear_smallm``), added in slice order; or a pair of float32 updates in either form, of which the second
+    is added behind the first."""
     rows, H = x.shape
+    second = None
+    if isinstance(delta, (tuple, list)):
+        _need(len(delta) == 2, "add_rmsnorm: one update or a pair")
+        delta, second = delta
+    _need_cuda(x, delta, second, weight, out)
     _need(x.dtype == torch.float32 and x.is_contiguous(), "add_rmsnorm: x must be contiguous float32")
     _need(weight.dtype == torch.float32 and weight.numel() == H, "add_rmsnorm: weight must be float32 [H]")
     _need(out.shape == x.shape and out.is_contiguous(), "add_rmsnorm: out shape")
-    partials, n_part, stride = None, 0, 0
-    if delta is not None and delta.dim() == 3:
-        _need(delta.dtype == torch.float32 and tuple(delta.shape[1:]) == (rows, H) and delta.is_contiguous(),
+
+    def slices(d):
+        n = d.shape[0] if d.dim() == 3 else 1
+        _need(d.dtype == torch.float32 and tuple(d.shape[-2:]) == (rows, H) and d.is_contiguous(),
               "add_rmsnorm: partial sums must be contiguous float32 [slices, rows, H]")
-        partials, n_part, stride, delta = delta, delta.shape[0], rows * H, None
+        return d, n, rows * H
+
+    p1, p2 = (None, 0, 0), (None, 0, 0)
+    if delta is not None and (delta.dim() == 3 or second is not None or (delta.dtype == torch.float32 and out.dtype != torch.float32)):
+        p1, delta = slices(delta), None
+        if second is not None:
+            p2 = slices(second)
     elif delta is not None:
         _need(delta.shape == x.shape and delta.dtype == out.dtype and delta.is_contiguous(), "add_rmsnorm: delta")
     f = _fn(_libs.get("elementwise.cu"), f"tkb_add_rmsnorm_{_suffix(out.dtype)}")
-    _check(f(_ptr(x), _ptr(delta), _ptr(partials), c_int(n_part), ctypes.c_longlong(stride), _ptr(weight), _ptr(out),
-             c_float(eps), c_int(rows), c_int(H), _stream()), "add_rmsnorm")
+    _check(f(_ptr(x), _ptr(delta), _ptr(p1[0]), c_int(p1[1]), ctypes.c_longlong(p1[2]), _ptr(p2[0]), c_int(p2[1]),
+             ctypes.c_longlong(p2[2]), _ptr(weight), _ptr(out), c_float(eps), c_int(rows), c_int(H), _stream()), "add_rmsnorm")
 
 
 def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor, page_indptr: torch.Tensor,
@@ -315,6 +326,19 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, interleave: int = 0, act:
     _need(gate_up.is_contiguous() and out.is_contiguous() and out.dtype == gate_up.dtype, "silu_mul: layout")
     f = _fn(_libs.get("elementwise.cu"), f"tkb_{act}_mul_{_suffix(out.dtype)}")
     _check(f(_ptr(gate_up), _ptr(out), c_int(rows), c_int(two_i // 2), c_int(interleave), _stream()), "silu_mul")
+
+
+def gelu_rows(z: torch.Tensor, out: torch.Tensor) -> None:
+    """out [rows, I] = gelu(z), the exact (erf) form; z [rows, I] in out's dtype or float32, or float32 slices
+    [slices, rows, I] of a split product, added in slice order."""
+    _need_cuda(z, out)
+    _need(z.is_contiguous() and out.is_contiguous() and tuple(z.shape[-2:]) == tuple(out.shape), "gelu_rows: shapes")
+    f32 = z.dtype == torch.float32
+    _need(f32 or (z.dtype == out.dtype and z.dim() == 2), "gelu_rows: z float32 or in out's type")
+    n = z.shape[0] if z.dim() == 3 else 1
+    _check(_fn(_libs.get("elementwise.cu"), f"tkb_gelu_rows_{_suffix(out.dtype)}")(
+        _ptr(z if f32 else None), c_int(n), ctypes.c_longlong(out.numel()), _ptr(None if f32 else z), _ptr(out),
+        ctypes.c_longlong(out.numel()), _stream()), "gelu_rows")
 
 
 def gather_rows(src: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
@@ -606,19 +630,20 @@ def can_use_tcgen05(a: torch.Tensor, w: torch.Tensor) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor, gated: bool = False) -> torch.Tensor:
+def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor, gated: bool = False, gelu: bool = False) -> torch.Tensor:
     """a[M, K] @ w[N, K]^T in bfloat16 on the tcgen05 tensor cores (TMA-fed, accumulator in tensor memory).
     ``gated``: ``w`` interleaves gate/up rows (``interleave_gate_up``); the result is silu(gate)*up [M, N/2].
+    ``gelu`` (ungated): the exact GELU of every result in the epilogue.
     ``status``: the device status word; a bounded wait that runs out sets its bit 4."""
     _need_cuda(a, w, status)
     _need(can_use_tcgen05(a, w), "gemm_tcgen05: bfloat16 operands, K and strides multiples of 8, 16-byte aligned")
     M, K = a.shape
     N = w.shape[0]
-    _need(w.shape[1] == K and (not gated or N % 16 == 0), "gemm_tcgen05: shapes")
+    _need(w.shape[1] == K and (not gated or N % 16 == 0) and not (gated and gelu), "gemm_tcgen05: shapes")
     out = torch.empty((M, N // 2 if gated else N), dtype=torch.bfloat16, device=a.device)
     _check(_fn(_libs.get("gemm_tcgen05.cu"), "tkb_gemm_tcgen05_bf16")(
         _ptr(a), c_int(a.stride(0)), _ptr(w), c_int(w.stride(0)), _ptr(out), c_int(out.stride(0)), c_int(M), c_int(N),
-        c_int(K), c_int(1 if gated else 0), _ptr(status), _stream()), "gemm_tcgen05")
+        c_int(K), c_int(1 if gated else (2 if gelu else 0)), _ptr(status), _stream()), "gemm_tcgen05")
     return out
 
 
@@ -954,7 +979,7 @@ def moe_route(h: torch.Tensor, router_w: torch.Tensor, router_b: torch.Tensor | 
     softmax over them (float32 [T, top]).  ``scored`` = dict(correction float32 [E] or None, groups, keep, scale): the
     other way of choosing: scores sigmoid(logits); the choice by score + correction among the experts of the best
     ``keep`` of ``groups`` equal groups of neighbours (a group scores the sum of its two largest choice scores); the
-    weights are the chosen scores over their sum, times ``scale``.
+    weights are the chosen scores over their sum, times ``scale`` (with ``renormalize`` False: the scores times ``scale``).
     ``over_all`` (the plain way of choosing): the weights are the chosen experts' shares of the softmax over ALL experts,
     not renormalised; ``scale`` multiplies the plain way's weights."""
     _need_cuda(h, router_w, router_b, token_seq, top_idx, top_w)
@@ -976,7 +1001,8 @@ def moe_route(h: torch.Tensor, router_w: torch.Tensor, router_b: torch.Tensor | 
         f = _fn(_libs.get("moe.cu"), f"tkb_moe_route_scored_{_suffix(h.dtype)}")
         _check(f(_ptr(h), _ptr(router_w), _ptr(router_b), _ptr(corr), _ptr(token_seq), _ptr(top_idx), _ptr(top_w),
                  _ptr(logits), c_int(T), c_int(H), c_int(E), c_int(top), c_int(groups), c_int(keep),
-                 c_float(float(scored.get("scale", 1.0))), _stream()), "moe_route")
+                 c_float(float(scored.get("scale", 1.0))), c_int(1 if scored.get("renormalize", True) else 0), _stream()),
+               "moe_route")
         return
     f = _fn(_libs.get("moe.cu"), f"tkb_moe_route_{_suffix(h.dtype)}")
     _check(f(_ptr(h), _ptr(router_w), _ptr(router_b), _ptr(token_seq), _ptr(top_idx), _ptr(top_w), _ptr(logits), c_int(T),
@@ -1021,24 +1047,33 @@ def moe_order(top_idx: torch.Tensor, n_experts: int, offsets: torch.Tensor, orde
         c_int(src_token.numel() if src_token is not None else 0), _stream()), "moe_order")
 
 
-def moe_gather(src: torch.Tensor, src_token: torch.Tensor, out: torch.Tensor) -> None:
-    """out[p] = src[src_token[p]], zeros where src_token[p] < 0."""
-    _need_cuda(src, src_token, out)
+def moe_gather(src: torch.Tensor, src_token: torch.Tensor, out: torch.Tensor, order: torch.Tensor | None = None,
+               pair_scale: torch.Tensor | None = None, place_scale: torch.Tensor | None = None) -> None:
+    """out[p] = src[src_token[p]], zeros where src_token[p] < 0.  ``place_scale`` float32 [places]: receives
+    pair_scale[order[p]] (0 at the padding)."""
+    _need_cuda(src, src_token, out, order, pair_scale, place_scale)
+    _need(place_scale is None or (order is not None and pair_scale is not None and pair_scale.dtype == torch.float32
+                                  and place_scale.dtype == torch.float32 and place_scale.numel() == out.shape[0]
+                                  and order.numel() >= out.shape[0]), "moe_gather: scales float32, a place each")
     _need(src.is_contiguous() and out.is_contiguous() and out.dtype == src.dtype and out.shape[1] == src.shape[1]
           and src_token.dtype == torch.int32 and src_token.numel() == out.shape[0], "moe_gather: shapes")
     f = _fn(_libs.get("moe.cu"), f"tkb_moe_gather_{_suffix(src.dtype)}")
-    _check(f(_ptr(src), _ptr(src_token), _ptr(out), c_int(out.shape[0]), c_int(src.shape[1]), _stream()), "moe_gather")
+    _check(f(_ptr(src), _ptr(src_token), _ptr(out), c_int(out.shape[0]), c_int(src.shape[1]), _ptr(order), _ptr(pair_scale),
+             _ptr(place_scale), _stream()), "moe_gather")
 
 
 def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, status: torch.Tensor,
-                         gated: bool = False, gelu: bool = False, clamp: tuple[float, float] | None = None) -> torch.Tensor:
+                         gated: bool = False, gelu: bool = False, clamp: tuple[float, float] | None = None,
+                         row_scale: torch.Tensor | None = None) -> torch.Tensor:
     """Row tile i (128 rows) of a[M, K] times the weights w[tile_group[i]] of w [groups, N, K], bfloat16 on the tcgen05
     tensor cores; tiles with tile_group[i] < 0 are left out (their rows of the result are not written).
     ``gated``: every group's rows interleave gate and up (``interleave_gate_up``); the result is [M, N / 2].
     ``gelu`` (ungated): the exact GELU of every result in the epilogue.  ``clamp`` = (limit, alpha), with ``gated``:
     the clamped unit g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), in the SiLU's
-    place."""
-    _need_cuda(a, w, tile_group, status)
+    place.  ``row_scale`` float32 [M] (``gated``, no ``clamp``): row i of ``a`` counts row_scale[i] times."""
+    _need_cuda(a, w, tile_group, status, row_scale)
+    _need(row_scale is None or (gated and clamp is None and row_scale.dtype == torch.float32 and row_scale.numel() >= a.shape[0]),
+          "gemm_tcgen05_grouped: row_scale float32 [M], with the SiLU-gated form")
     G, N, K = w.shape
     _need(can_use_tcgen05(a, w.view(G * N, K)) and a.shape[1] == K, "gemm_tcgen05_grouped: bfloat16, K a multiple of 8")
     M = a.shape[0]
@@ -1054,18 +1089,23 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Ten
         return out
     _check(_fn(_libs.get("gemm_tcgen05.cu"), "tkb_gemm_tcgen05_grouped_bf16")(
         _ptr(a), c_int(a.stride(0)), _ptr(w), c_int(K), _ptr(out), c_int(out.stride(0)), c_int(M), c_int(N), c_int(K),
-        c_int(1 if gated else (2 if gelu else 0)), _ptr(tile_group), c_int(G), _ptr(status), _stream()), "gemm_tcgen05_grouped")
+        c_int(1 if gated else (2 if gelu else 0)), _ptr(tile_group), c_int(G), _ptr(row_scale), _ptr(status), _stream()),
+        "gemm_tcgen05_grouped")
     return out
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor | None,
-             top: int, gated: bool, gelu: bool = False, clamp: tuple[float, float] | None = None) -> None:
+             top: int, gated: bool, gelu: bool = False, clamp: tuple[float, float] | None = None,
+             pair_scale: torch.Tensor | None = None) -> None:
     """The experts' products over the ordering.  w [E, N (2N if gated), K]; a [., K]; row p of ``out`` is made from
     row order[p] // top of ``a`` (row p if ``order`` is None) with the weights of the expert whose span holds p.
     gated: out = silu(a w_gate^T) * (a w_up^T) in a's type [places, N]; gelu: out = gelu(a w^T) (exact) in a's type;
     else float32 [places, N].  ``clamp`` = (limit, alpha), with ``gated``: the clamped unit
-    g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), in the SiLU's place."""
-    _need_cuda(a, w, out, offsets, order)
+    g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), in the SiLU's place.
+    ``pair_scale`` float32 [pairs] (``gated``, no ``clamp``, with ``order``): the row of pair order[p] counts so many times."""
+    _need_cuda(a, w, out, offsets, order, pair_scale)
+    _need(pair_scale is None or (gated and clamp is None and order is not None and pair_scale.dtype == torch.float32
+                                 and pair_scale.is_contiguous() and pair_scale.numel() == out.shape[0]), "moe_gemm: pair_scale float32 [pairs]")
     _need(clamp is None or (gated and clamp[0] > 0), "moe_gemm: the clamped unit is a gated form with a positive limit")
     E, NN, K = w.shape
     N = NN // 2 if gated else NN
@@ -1078,14 +1118,15 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch
             c_int(out.shape[0]), c_int(E), c_int(N), c_int(K), c_float(clamp[0]), c_float(clamp[1]), _stream()), "moe_gemm")
         return
     name = f"tkb_moe_gemm_{'gated_' if gated else ('gelu_' if gelu else '')}{_suffix(a.dtype)}"
+    extra = (_ptr(pair_scale),) if gated else ()
     _check(_fn(_libs.get("moe.cu"), name)(_ptr(a), c_int(a.stride(0)), _ptr(w), _ptr(out), c_int(out.stride(0)),
                                           _ptr(offsets), _ptr(order), c_int(top), c_int(out.shape[0]), c_int(E), c_int(N),
-                                          c_int(K), _stream()), "moe_gemm")
+                                          c_int(K), *extra, _stream()), "moe_gemm")
 
 
 def moe_combine(y: torch.Tensor, place_of: torch.Tensor, top_w: torch.Tensor, shared: torch.Tensor | None,
-                out: torch.Tensor, shared_gate: torch.Tensor | None = None) -> None:
-    """out[t] = sum_k top_w[t, k] * y[place_of[t, k]] (+ shared[t]); y float32 [places, H]; shared [T, H] in out's type
+                out: torch.Tensor, shared_gate: torch.Tensor | None = None, weigh: bool = True) -> None:
+    """out[t] = sum_k top_w[t, k] * y[place_of[t, k]] (+ shared[t]) (``weigh`` False: without the factors top_w); y float32 [places, H]; shared [T, H] in out's type
     or float32 slices [slices, T, H].  ``shared_gate`` float32 [T]: the shared part counts sigmoid(shared_gate[t])
     times."""
     _need_cuda(y, place_of, top_w, shared, out, shared_gate)
@@ -1098,7 +1139,7 @@ def moe_combine(y: torch.Tensor, place_of: torch.Tensor, top_w: torch.Tensor, sh
     d, sl, n_sl, stride = _split_update(shared, T, H, out.dtype, "moe_combine")
     f = _fn(_libs.get("moe.cu"), f"tkb_moe_combine_y16_{_suffix(out.dtype)}" if y.dtype == torch.bfloat16
             else f"tkb_moe_combine_{_suffix(out.dtype)}")
-    _check(f(_ptr(y), _ptr(place_of), _ptr(top_w), _ptr(d), _ptr(sl), c_int(n_sl), ctypes.c_longlong(stride), _ptr(out),
+    _check(f(_ptr(y), _ptr(place_of), _ptr(top_w if weigh else None), _ptr(d), _ptr(sl), c_int(n_sl), ctypes.c_longlong(stride), _ptr(out),
              c_int(T), c_int(H), c_int(top), _ptr(shared_gate), _stream()), "moe_combine")
 
 
@@ -1306,14 +1347,17 @@ def ssm_prep(proj: torch.Tensor, xbc_off: int, channels: int, conv_w: torch.Tens
 def decay_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, heads_per_qk: int, dt_dec: torch.Tensor | None,
                decay_head: torch.Tensor | None, skip: torch.Tensor | None, state: torch.Tensor, out: torch.Tensor,
                seq_slot: torch.Tensor, seq_q_start: torch.Tensor, seq_q_len: torch.Tensor, n_seqs: int, heads: int,
-               dim: int, vdim: int, write_state: bool = True, decay_vec: torch.Tensor | None = None) -> None:
+               dim: int, vdim: int, write_state: bool = True, decay_vec: torch.Tensor | None = None,
+               ones_out: torch.Tensor | None = None) -> None:
     """S_t = a_t S_(t-1) + (c_t k_t) v_t^T, o_t = S_t^T q_t + skip * v_t over each request's tokens.  q, k [T, . * dim]
     and v [T, heads * vdim] are float32 (column slices allowed); head h reads q and k number h // heads_per_qk.
     ``dt_dec`` [T, 2 heads] = (c, a) per token, or ``decay_head`` [heads] with
     c = 1, or ``decay_vec`` float32 [T, heads * dim] (a column slice allowed): a decay for every key channel,
     S_t = diag(f_t) S_(t-1) + k_t v_t^T.  state float32 [slots, n], S^T of the heads first: [heads, vdim, dim]; out
-    float32 [T, heads * vdim]."""
-    _need_cuda(q, k, v, dt_dec, decay_head, skip, state, out, seq_slot, seq_q_start, seq_q_len, decay_vec)
+    float32 [T, heads * vdim].  ``ones_out`` float32 [T, heads] (not with ``decay_vec``): a head's state holds one more
+    column, [heads, vdim + 1, dim], whose value is 1 at every token; its S^T q goes there."""
+    _need_cuda(q, k, v, dt_dec, decay_head, skip, state, out, seq_slot, seq_q_start, seq_q_len, decay_vec, ones_out)
+    vall = vdim + (1 if ones_out is not None else 0)
     T = q.shape[0]
     for t in (q, k, v):
         _need(t.dtype == torch.float32 and t.stride(1) == 1 and t.shape[0] == T, "decay_walk: float32 rows")
@@ -1327,16 +1371,92 @@ def decay_walk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, heads_per_qk: 
           "decay_walk: dt_dec float32 [T, 2 heads]")
     for t in (decay_head, skip):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == heads), "decay_walk: float32 [heads]")
-    _need(state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] >= heads * vdim * dim,
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] >= heads * vall * dim,
           "decay_walk: state float32 [slots, n]")
+    _need(ones_out is None or (decay_vec is None and ones_out.dtype == torch.float32 and ones_out.is_contiguous()
+                               and tuple(ones_out.shape) == (T, heads)), "decay_walk: ones_out float32 [T, heads]")
     _need(out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (T, heads * vdim), "decay_walk: out float32 [T, heads * vdim]")
-    defines = _walk_defines(dim, vdim, n_seqs * heads * vdim, T == n_seqs, q.device)
+    defines = _walk_defines(dim, vdim, n_seqs * heads * vall, T == n_seqs, q.device)
     _check(_fn(_libs.get("decay_recurrence.cu", **defines), "tkb_decay_walk")(
         _ptr(q), c_int(q.stride(0)), _ptr(k), c_int(k.stride(0)), c_int(heads_per_qk), _ptr(decay_vec),
         c_int(decay_vec.stride(0) if decay_vec is not None else 0), _ptr(v), c_int(v.stride(0)),
         _ptr(dt_dec), _ptr(decay_head), _ptr(skip), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(out),
         _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), c_int(n_seqs), c_int(T), c_int(heads), c_int(dim), c_int(vdim),
-        c_int(1 if write_state else 0), _stream()), "decay_walk")
+        c_int(1 if write_state else 0), _ptr(ones_out), _stream()), "decay_walk")
+
+
+def memory_gates(proj: torch.Tensor, i_off: int, f_off: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+                 state: torch.Tensor, m_off: int, seq_slot: torch.Tensor, seq_q_start: torch.Tensor, seq_q_len: torch.Tensor,
+                 n_seqs: int, dt_dec: torch.Tensor, floor: torch.Tensor, defines: dict, write_state: bool = True) -> None:
+    """Gates of a matrix memory from float32 projections [T, .]: i = cap tanh((proj[:, i_off + h] + i_bias[h]) / cap),
+    f = log_sigmoid(cap tanh((proj[:, f_off + h] + f_bias[h]) / cap)), m_t = max(f_t + m_(t-1), i_t) with m from and to
+    state[slot, m_off + h]; dt_dec [T, 2 heads] receives exp(i - m_t), then exp(f + m_(t-1) - m_t); floor [T, heads]
+    receives exp(-m_t)."""
+    _need_cuda(proj, i_bias, f_bias, state, seq_slot, seq_q_start, seq_q_len, dt_dec, floor)
+    T, heads = floor.shape
+    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == T and proj.shape[1] >= max(i_off, f_off) + heads,
+          "memory_gates: float32 projections")
+    for v in (i_bias, f_bias):
+        _need(v.dtype == torch.float32 and v.is_contiguous() and v.numel() == heads, "memory_gates: float32 [heads] biases")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] >= m_off + heads
+          and cap > 0, "memory_gates: state float32 [slots, n], a positive cap")
+    _need(dt_dec.dtype == torch.float32 and dt_dec.is_contiguous() and tuple(dt_dec.shape) == (T, 2 * heads)
+          and floor.dtype == torch.float32 and floor.is_contiguous(), "memory_gates: dt_dec [T, 2 heads], floor [T, heads]")
+    _check(_fn(_libs.get("decay_recurrence.cu", **defines), "tkb_memory_gates")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(i_off), c_int(f_off), _ptr(i_bias), _ptr(f_bias), c_float(cap), _ptr(state),
+        ctypes.c_longlong(state.stride(0)), ctypes.c_longlong(m_off), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len),
+        c_int(n_seqs), c_int(heads), _ptr(dt_dec), _ptr(floor), c_int(1 if write_state else 0), _stream()), "memory_gates")
+
+
+def memory_norm(raw: torch.Tensor, den: torch.Tensor, floor: torch.Tensor, gate: torch.Tensor, g_off: int, weight: torch.Tensor,
+                q_scale: float, den_eps: float, eps: float, out_scale: float, out: torch.Tensor, heads: int, vdim: int,
+                defines: dict) -> None:
+    """out[t] = N(o) * weight * sigmoid(gate[t, g_off:]) * out_scale, head by head, with
+    o = q_scale * raw / (max(|q_scale * den|, floor) + den_eps) and N the division by the head's root mean square; raw
+    float32 [T, heads * vdim], den and floor float32 [T, heads]; ``out`` may be a column slice of a wider tensor."""
+    _need_cuda(raw, den, floor, gate, weight, out)
+    T = raw.shape[0]
+    _need(raw.dtype == torch.float32 and raw.is_contiguous() and raw.shape[1] == heads * vdim, "memory_norm: raw float32 [T, heads * vdim]")
+    for v in (den, floor):
+        _need(v.dtype == torch.float32 and v.is_contiguous() and tuple(v.shape) == (T, heads), "memory_norm: float32 [T, heads]")
+    _need(gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == T and gate.shape[1] >= g_off + heads * vdim,
+          "memory_norm: float32 gate columns")
+    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == heads * vdim, "memory_norm: weight float32")
+    _need(tuple(out.shape) == (T, heads * vdim) and out.stride(1) == 1, "memory_norm: out")
+    _check(_fn(_libs.get("decay_recurrence.cu", **defines), f"tkb_memory_norm_{_suffix(out.dtype)}")(
+        _ptr(raw), _ptr(den), _ptr(floor), _ptr(gate), c_int(gate.stride(0)), c_int(g_off), _ptr(weight), c_float(q_scale),
+        c_float(den_eps), c_float(eps), c_float(out_scale), _ptr(out), c_int(_row_stride(out)), c_int(heads), c_int(vdim),
+        c_int(T), _stream()), "memory_norm")
+
+
+def real_gated_recurrence(proj: torch.Tensor, y_off: int, x_off: int, y_bias: torch.Tensor, x_bias: torch.Tensor,
+                          taps: torch.Tensor, conv_bias: torch.Tensor, w_r: torch.Tensor, b_r: torch.Tensor, w_i: torch.Tensor,
+                          b_i: torch.Tensor, neg: torch.Tensor, state: torch.Tensor, token_seq: torch.Tensor,
+                          seq_slot: torch.Tensor, seq_q_start: torch.Tensor, seq_q_len: torch.Tensor, out: torch.Tensor,
+                          write_state: bool = True) -> None:
+    """Griffin's recurrent block between its projections (csrc/gated_recurrence.cu).  proj float32 [T, .] holds W_y h at
+    column ``y_off`` and W_x h at ``x_off``, C columns each; taps float32 [C, K]; w_r, w_i [parts, C / parts, C / parts] in
+    out's dtype; neg float32 [C] = -decay_scale * softplus(lam); state float32 [slots, >= C * K]: S, then the convolution's
+    last K - 1 inputs; out [T, C] = S_t * gelu_tanh(y_t)."""
+    _need_cuda(proj, y_bias, x_bias, taps, conv_bias, w_r, b_r, w_i, b_i, neg, state, token_seq, seq_slot, seq_q_start, seq_q_len, out)
+    T, C = out.shape
+    K, parts = taps.shape[1], w_r.shape[0]
+    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == T and proj.shape[1] >= max(y_off, x_off) + C,
+          "real_gated_recurrence: float32 projections")
+    for v, what in ((y_bias, "y"), (x_bias, "x"), (conv_bias, "convolution"), (b_r, "r"), (b_i, "i"), (neg, "decay")):
+        _need(v.dtype == torch.float32 and v.is_contiguous() and v.numel() == C, f"real_gated_recurrence: {what} vector float32 [C]")
+    _need(taps.dtype == torch.float32 and taps.is_contiguous() and taps.shape[0] == C, "real_gated_recurrence: taps float32 [C, K]")
+    _need(C % parts == 0 and w_r.dtype == w_i.dtype == out.dtype and w_r.is_contiguous() and w_i.is_contiguous()
+          and tuple(w_r.shape) == tuple(w_i.shape) == (parts, C // parts, C // parts), "real_gated_recurrence: gate matrices [parts, n, n]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] >= C * K,
+          "real_gated_recurrence: state float32 [slots, C * K]")
+    _need(out.is_contiguous() and token_seq.dtype == torch.int32 and token_seq.numel() >= T, "real_gated_recurrence: out, token_seq")
+    scratch = torch.empty((2, T, C), dtype=torch.float32, device=out.device)
+    _check(_fn(_libs.get("gated_recurrence.cu"), f"tkb_rglru_{_suffix(out.dtype)}")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(y_off), c_int(x_off), _ptr(y_bias), _ptr(x_bias), _ptr(taps), _ptr(conv_bias),
+        c_int(K), c_int(C), c_int(parts), _ptr(w_r), _ptr(b_r), _ptr(w_i), _ptr(b_i), _ptr(neg), _ptr(state),
+        ctypes.c_longlong(state.stride(0)), _ptr(token_seq), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), c_int(T),
+        _ptr(scratch[0]), _ptr(scratch[1]), _ptr(out), c_int(1 if write_state else 0), _stream()), "real_gated_recurrence")
 
 
 def gla_gates(proj: torch.Tensor, low_off: int, rank: int, a2t: torch.Tensor, bias: torch.Tensor | None, tau: float,
@@ -1386,9 +1506,9 @@ def silu_cols(x: torch.Tensor, ncols: int, defines: dict) -> None:
 
 # ---------------------------------------------------------------------------------------------
 # Attention with a score cap and a sink, keys and values of different sizes (csrc/attention_sink.cu)
-def sink_attention_defines(dim: int, vdim: int, sigmoid: bool = False, maps: int = 1) -> dict:
+def sink_attention_defines(dim: int, vdim: int, sigmoid: bool = False, maps: int = 1, distance: bool = False) -> dict:
     """``sigmoid``: the build whose weights are sigmoid(score), not a softmax.  ``maps``: attention maps a head (each
-    with query and key vectors of its own, over the same values)."""
+    with query and key vectors of its own, over the same values).  ``distance``: the build with a bias by distance."""
     _need(0 < dim <= 512 and 0 < vdim <= 512, f"sink attention: head sizes up to 512, not {dim} / {vdim}")
     _need(1 <= maps <= 4, f"sink attention: one to four maps a head, not {maps}")
     d = dict(TKB_QK=dim, TKB_VD=vdim)
@@ -1396,6 +1516,8 @@ def sink_attention_defines(dim: int, vdim: int, sigmoid: bool = False, maps: int
         d["TKB_SIGMOID"] = 1
     if maps > 1:
         d["TKB_MAPS"] = maps
+    if distance:
+        d["TKB_DIST"] = 1
     return d
 
 
@@ -1404,14 +1526,14 @@ def sink_attn_prep(qkv: torch.Tensor, bias: torch.Tensor | None, unit_norm: bool
                    page_ids: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, vdim: int, page_size: int,
                    write_cache: bool, status: torch.Tensor, norm_w: torch.Tensor | None = None,
                    rot_freq: torch.Tensor | None = None, rot_dims: int = 0, rot_pairs: bool = False,
-                   values_are_keys: bool = False, sigmoid: bool = False, maps: int = 1) -> None:
+                   values_are_keys: bool = False, sigmoid: bool = False, maps: int = 1, distance: bool = False) -> None:
     """qkv float32 [T, heads*maps*dim | kv heads*maps*dim | kv heads*vdim | anything else] -> (+ bias, q and k vectors
     divided by their root mean square) q_out [T, heads*maps*dim] and the tokens' [k of every map | v] rows in cache
     [pages, kv heads, page_size, maps*dim + vdim].
     ``norm_w`` float32 [2, dim]: weights of the q heads' and the k heads' norm.  ``rot_freq`` float64 [rot_dims / 2]:
     q and k are rotated by position on their first ``rot_dims`` channels (``rot_pairs``: channel 2i with 2i + 1, else
     i with i + rot_dims / 2).  ``values_are_keys``: the projections hold no v; a token's value is its key as projected
-    (before norm and rotation).  ``sigmoid``: the kernel build of the sigmoid form."""
+    (before norm and rotation).  ``sigmoid``, ``distance``: the kernel build that the attention itself uses."""
     _need_cuda(qkv, bias, q_out, cache, positions, token_seq, page_indptr, page_ids, status, norm_w, rot_freq)
     T = qkv.shape[0]
     C = (n_heads + n_kv_heads) * maps * dim + (0 if values_are_keys else n_kv_heads * vdim)
@@ -1425,12 +1547,17 @@ def sink_attn_prep(qkv: torch.Tensor, bias: torch.Tensor | None, unit_norm: bool
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == C), "sink_attn_prep: bias float32")
     _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, n_heads * maps * dim) and q_out.dtype == cache.dtype, "sink_attn_prep: q_out")
     _need(cache.is_contiguous() and tuple(cache.shape[1:]) == (n_kv_heads, page_size, maps * dim + vdim), "sink_attn_prep: cache rows")
-    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps)), f"tkb_sink_attn_prep_{_suffix(cache.dtype)}")(
+    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, distance)), f"tkb_sink_attn_prep_{_suffix(cache.dtype)}")(
         _ptr(qkv), c_int(qkv.stride(0)), _ptr(bias), c_int(1 if unit_norm else 0), c_float(eps), _ptr(q_out), _ptr(cache),
         _ptr(positions), _ptr(token_seq), _ptr(page_indptr), _ptr(page_ids), c_int(T), c_int(n_heads), c_int(n_kv_heads),
         c_int(page_size), c_int(cache.shape[0]), c_int(1 if write_cache else 0), _ptr(status), _ptr(norm_w), _ptr(rot_freq),
         c_int(rot_dims if rot_freq is not None else 0), c_int(1 if rot_pairs else 0), c_int(1 if values_are_keys else 0),
         _stream()), "sink_attn_prep")
+
+
+def _row_stride(t: torch.Tensor) -> int:
+    """The row stride of a 2-D tensor (its width where there is one row: torch reports any stride there)."""
+    return t.stride(0) if t.shape[0] > 1 else max(t.stride(0), t.shape[1])
 
 
 def _head_vectors(n_heads: int, what: str, *vectors):
@@ -1440,8 +1567,8 @@ def _head_vectors(n_heads: int, what: str, *vectors):
 
 def _sink_out_ok(out: torch.Tensor, rows: int, n_heads: int, vdim: int, maps: int, act: torch.dtype) -> bool:
     """One map: [rows, heads * vdim] in the activation type.  Several: float32 [rows, heads * maps * vdim], the maps'
-    outputs side by side, unrounded."""
-    return (out.is_contiguous() and tuple(out.shape) == (rows, n_heads * maps * vdim)
+    outputs side by side, unrounded.  Rows may be part of wider ones."""
+    return (out.stride(1) == 1 and tuple(out.shape) == (rows, n_heads * maps * vdim)
             and out.dtype == (act if maps == 1 else torch.float32))
 
 
@@ -1450,24 +1577,28 @@ def attn_sink(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, token_seq
               sinks: torch.Tensor | None, n_heads: int, n_kv_heads: int, dim: int, vdim: int, page_size: int,
               scale: float, softcap: float | None, window: int | None, status: torch.Tensor,
               head_scale: torch.Tensor | None = None, head_bias: torch.Tensor | None = None, sigmoid: bool = False,
-              maps: int = 1, keep_first: int = 0) -> None:
+              maps: int = 1, keep_first: int = 0, chunk: int | None = None, head_slope: torch.Tensor | None = None,
+              out_scale: float = 1.0) -> None:
     """Attention of ``n_rows`` tokens (``rows`` names them; None: all) over their requests' cached [k | v] rows.
     ``head_scale`` / ``head_bias`` float32 [heads]: a factor on a head's scale, a number added to its scores.
     ``sigmoid``: weights sigmoid(score) instead of a softmax (no sink).  ``maps`` > 1: so many attention maps a head,
     each a softmax of its own; ``out`` then is float32 [rows, heads * maps * vdim].  ``keep_first``: with a window, the
-    request's first so many positions stay visible."""
-    _need_cuda(q, out, cache, token_seq, positions, page_indptr, page_ids, rows, sinks, status, head_scale, head_bias)
-    _head_vectors(n_heads * maps, "attn_sink", head_scale, head_bias)
+    request's first so many positions stay visible.  ``chunk``: a query sees the keys of its own chunk of so many positions
+    only.  ``head_slope`` float32 [heads]: a slope times the distance comes off a head's scores.  ``out_scale`` multiplies
+    the result; ``out`` may be a column slice of a wider tensor."""
+    _need_cuda(q, out, cache, token_seq, positions, page_indptr, page_ids, rows, sinks, status, head_scale, head_bias, head_slope)
+    _head_vectors(n_heads * maps, "attn_sink", head_scale, head_bias, head_slope)
     _need(not (sigmoid and sinks is not None), "attn_sink: the sigmoid form has no sink")
     _need(q.is_contiguous() and q.shape[1] == n_heads * maps * dim and q.dtype == cache.dtype
           and _sink_out_ok(out, n_rows, n_heads, vdim, maps, cache.dtype), "attn_sink: q and out")
     _need(cache.is_contiguous() and tuple(cache.shape[1:]) == (n_kv_heads, page_size, maps * dim + vdim), "attn_sink: cache rows")
     _need(sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == n_heads * maps), "attn_sink: sinks float32 [heads]")
-    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps)), f"tkb_attn_sink_simt_{_suffix(cache.dtype)}")(
+    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, head_slope is not None)), f"tkb_attn_sink_simt_{_suffix(cache.dtype)}")(
         _ptr(q), _ptr(out), _ptr(cache), _ptr(token_seq), _ptr(positions), _ptr(page_indptr), _ptr(page_ids), _ptr(rows),
         c_int(n_rows), _ptr(sinks), c_int(n_heads), c_int(n_kv_heads), c_int(page_size), c_float(scale),
-        c_float(softcap or 0.0), c_int(window or 0), c_int(keep_first if window else 0), c_int(cache.shape[0]),
-        _ptr(status), _ptr(head_scale), _ptr(head_bias), _stream()), "attn_sink")
+        c_float(softcap or 0.0), c_int(window or 0), c_int(keep_first if window else 0), c_int(chunk or 0),
+        c_int(cache.shape[0]), _ptr(status), _ptr(head_scale), _ptr(head_bias), _ptr(head_slope), c_int(_row_stride(out)),
+        c_float(out_scale), _stream()), "attn_sink")
 
 
 def can_use_attn_sink_tc(dtype: torch.dtype, dim: int, vdim: int, maps: int = 1) -> bool:
@@ -1481,12 +1612,13 @@ def attn_sink_tc(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, seq_q_
                  sinks: torch.Tensor | None, n_heads: int, n_kv_heads: int, dim: int, vdim: int, page_size: int, scale: float,
                  softcap: float | None, window: int | None, status: torch.Tensor, portions: bool = True,
                  singles: bool = True, head_scale: torch.Tensor | None = None, head_bias: torch.Tensor | None = None,
-                 sigmoid: bool = False, maps: int = 1, keep_first: int = 0) -> None:
+                 sigmoid: bool = False, maps: int = 1, keep_first: int = 0, chunk: int | None = None,
+                 head_slope: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
     """Attention of every token of the step on the tensor cores (bfloat16): out [T, heads * vdim] (``maps`` > 1: float32
     [T, heads * maps * vdim]).  ``portions`` / ``singles``: whether the step can hold requests with several tokens /
-    with one (a kernel each).  ``keep_first``: as in ``attn_sink``."""
-    _need_cuda(q, out, cache, seq_q_start, seq_q_len, seq_kv_len, page_indptr, page_ids, sinks, status, head_scale, head_bias)
-    _head_vectors(n_heads * maps, "attn_sink_tc", head_scale, head_bias)
+    with one (a kernel each).  ``keep_first``, ``chunk``, ``head_slope``, ``out_scale``: as in ``attn_sink``."""
+    _need_cuda(q, out, cache, seq_q_start, seq_q_len, seq_kv_len, page_indptr, page_ids, sinks, status, head_scale, head_bias, head_slope)
+    _head_vectors(n_heads * maps, "attn_sink_tc", head_scale, head_bias, head_slope)
     _need(not (sigmoid and sinks is not None), "attn_sink_tc: the sigmoid form has no sink")
     T = q.shape[0]
     _need(can_use_attn_sink_tc(cache.dtype, dim, vdim, maps), "attn_sink_tc: bfloat16 rows, key and value sizes multiples of 16")
@@ -1502,16 +1634,16 @@ def attn_sink_tc(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, seq_q_
 
         blocks = n_seqs * n_kv_heads * ((n_heads // n_kv_heads + 15) // 16)  # (a block serves every map of its heads)
         splits = max(1, min(8, (2 * device_limits(q.device).sm_count) // max(1, blocks)))
-        if window:
-            splits = min(splits, max(1, (window + 63) // 64))
+        if window or chunk:
+            splits = min(splits, max(1, (min(w for w in (window, chunk) if w) + 63) // 64))
         if splits > 1:
             part = torch.empty((n_seqs * n_heads * maps * splits * (vdim + 2),), dtype=torch.float32, device=q.device)
-    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps)), "tkb_attn_sink_tc_bf16")(
+    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, head_slope is not None)), "tkb_attn_sink_tc_bf16")(
         _ptr(q), _ptr(out), _ptr(cache), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(page_indptr),
         _ptr(page_ids), c_int(T), c_int(n_seqs), c_int(1 if portions else 0), c_int(1 if singles else 0), _ptr(sinks),
         c_int(n_heads), c_int(n_kv_heads), c_int(page_size), c_float(scale), c_float(softcap or 0.0), c_int(window or 0),
-        c_int(keep_first if window else 0), c_int(cache.shape[0]), _ptr(status), _ptr(part), c_int(splits), _ptr(head_scale),
-        _ptr(head_bias), _stream()), "attn_sink_tc")
+        c_int(keep_first if window else 0), c_int(chunk or 0), c_int(cache.shape[0]), _ptr(status), _ptr(part), c_int(splits),
+        _ptr(head_scale), _ptr(head_bias), _ptr(head_slope), c_int(_row_stride(out)), c_float(out_scale), _stream()), "attn_sink_tc")
 
 
 def diff_combine(a: torch.Tensor, lam: torch.Tensor, eps: float, mult: float, gate: torch.Tensor | None, gate_off: int,

@@ -47,13 +47,24 @@ class PagedCacheNeed:
     """Per-token keys and values kept in pages.  ``window``: only the last ``window`` keys
     (the query's own included) are ever read, so pages behind it can be given back.  ``planes``: 2 for keys and
     values, 1 for a mixer that keeps one row a token (a latent from which it makes both).  ``keep_first``: with a
-    window, the request's first so many keys are read by every later query too: their pages stay."""
+    window, the request's first so many keys are read by every later query too: their pages stay.  ``chunked``: the
+    window does not slide; the sequence is cut into chunks of ``window`` positions, counted from position 0, and a query
+    reads the keys of its own chunk only (never more than the sliding window would let it see)."""
 
     n_kv_heads: int
     head_dim: int
     window: int | None = None
     planes: int = 2
     keep_first: int = 0
+    chunked: bool = False
+
+    def first_visible(self, position: int) -> int:
+        """The first key that a query at ``position`` or any later one reads (kept first keys aside)."""
+        if not self.window:
+            return 0
+        if self.chunked:
+            return position // self.window * self.window
+        return max(0, position - self.window + 1)
 
 
 @dataclass(frozen=True)
@@ -116,6 +127,15 @@ class Mixer(Part):
     def cache_need(self) -> PagedCacheNeed | StateNeed | None:
         return None
 
+    def side_needs(self) -> dict:
+        """{name: need} of cache entries that the mixer holds beside ``cache_need()`` (a mixer made of several).  A mixer
+        that names some takes their caches in ``forward(..., side={name: cache})``."""
+        return {}
+
+    def inner_mixers(self) -> tuple:
+        """The mixers that this one is made of (itself, for a simple one)."""
+        return (self,)
+
     def plan_key(self):
         """A hashable key if this mixer wants a host-side work plan for each step, else None.  Mixers
         with equal keys share one plan."""
@@ -161,7 +181,8 @@ class InputStage(Part):
 class ResidualStream:
     """The running sum of a token's representation, held in float32, plus one pending
     update in the engine's dtype that the next norm adds before it normalises (so the add
-    costs no extra pass over memory).  ``h``: the same rows as ``x`` in the activation type, if the kernel that made
+    costs no extra pass over memory).  The update may also be float32 slices of a split product, or (norms that
+    take them) a pair of float32 updates, of the two sublayers of a block that read one norm.  ``h``: the same rows as ``x`` in the activation type, if the kernel that made
     ``x`` wrote them too (blocks whose sublayers read the stream itself)."""
 
     __slots__ = ("x", "delta", "h")
@@ -170,3 +191,11 @@ class ResidualStream:
         self.x = x
         self.delta = delta
         self.h = h
+
+    def settled(self) -> "torch.Tensor":
+        """A copy of the rows with the pending update added (for looking at a model layer by layer)."""
+        x = self.x.clone()
+        for d in (self.delta if isinstance(self.delta, (tuple, list)) else (self.delta,)):
+            if d is not None:
+                x += d.sum(0) if d.dim() == 3 else d
+        return x

@@ -15,6 +15,18 @@ from tokasaurus_b200.kernels import ops
 from tokasaurus_b200.parts.base import FeedForward, InputStage, Mixer, Norm, Part, ResidualStream
 
 
+def _side_needs(mixer: Mixer) -> dict:
+    return dict(mixer.side_needs()) if hasattr(mixer, "side_needs") else {}
+
+
+def _mix(mixer: Mixer, ctx, h, cache, out_rows, state: dict | None):
+    """``mixer.forward``, with the caches of its further entries if it names some."""
+    names = _side_needs(mixer)
+    if names:
+        return mixer.forward(ctx, h, cache, out_rows, side={n: (state or {}).get(n) for n in names})
+    return mixer.forward(ctx, h, cache, out_rows)
+
+
 class PreNormBlock(Part):
     def __init__(self, mixer_norm: Norm, mixer: Mixer, ffn_norm: Norm | None, ffn: FeedForward | None,
                  mixer_stage: InputStage | None = None, ffn_stage: InputStage | None = None):
@@ -50,6 +62,7 @@ class PreNormBlock(Part):
             need = stage.state_need() if stage is not None else None
             if need is not None:
                 out[name] = need
+        out.update(_side_needs(self.mixer))
         return out
 
     @staticmethod
@@ -71,7 +84,7 @@ class PreNormBlock(Part):
         cut_late = self.ffn_stage is not None and out_rows is not None
         if out_rows is not None and not cut_late:
             stream = self._cut(stream, out_rows)
-        stream.delta = self.mixer.forward(ctx, h, cache, None if cut_late else out_rows)
+        stream.delta = _mix(self.mixer, ctx, h, cache, None if cut_late else out_rows, stage_state)
         if self.ffn is None:
             return stream
         h = self._staged(ctx, self.ffn_norm, self.ffn_stage, stream, stage_state.get("ffn_stage"))
@@ -88,6 +101,49 @@ class PreNormBlock(Part):
         x = torch.empty((rows.numel(), stream.x.shape[1]), dtype=stream.x.dtype, device=stream.x.device)
         ops.gather_rows(stream.x, rows, x)
         return ResidualStream(x)
+
+
+class ParallelBlock(Part):
+    """A block whose mixer and feed-forward read ONE norm and whose outputs are added together:
+
+        h = norm(x),      x <- x + (mixer(h) + ffn(h))
+
+    The sublayers leave float32 updates (rows, or the slices of a K-split product); the pair stays pending and the next
+    norm adds both on its way (``parts.norm.RMSNorm``).  ``ffn=None``: the block is its mixer alone."""
+
+    def __init__(self, norm: Norm, mixer: Mixer, ffn: FeedForward | None):
+        self.norm, self.mixer, self.ffn = norm, mixer, ffn
+
+    def parts(self):
+        return tuple(p for p in (self.norm, self.mixer, self.ffn) if p is not None)
+
+    def weight_specs(self):
+        return tuple(s for p in self.parts() for s in p.weight_specs())
+
+    def kernel_modules(self, dtype):
+        return tuple(m for p in self.parts() for m in p.kernel_modules(dtype))
+
+    def bind(self, weights, rt) -> None:
+        for p in self.parts():
+            p.bind(weights, rt)
+
+    def state_needs(self) -> dict:
+        return _side_needs(self.mixer)
+
+    def forward(self, ctx, stream: ResidualStream, cache, out_rows=None, stage_state=None) -> ResidualStream:
+        h = self.norm.forward(ctx, stream)
+        if out_rows is not None:
+            stream = PreNormBlock._cut(stream, out_rows)
+        mixed = _mix(self.mixer, ctx, h, cache, out_rows, stage_state)
+        if self.ffn is None:
+            stream.delta = mixed
+            return stream
+        if out_rows is not None:
+            hc = torch.empty((out_rows.numel(), h.shape[1]), dtype=h.dtype, device=h.device)
+            ops.gather_rows(h, out_rows, hc)
+            h = hc
+        stream.delta = (mixed, self.ffn.forward(ctx, h))
+        return stream
 
 
 class OutputNormBlock(Part):

@@ -57,6 +57,8 @@ class GatedMLP(FeedForward):
             return ops.linear_out_f32(act, self.w_down, status) if self.out_f32 else ops.linear(act, self.w_down)
         if self.interleave and ops.can_use_few_rows(h, self.w_gate_up) and self.w_gate_up.shape[0] % 16 == 0:
             act = ops.linear_few_rows_gated(h, self.w_gate_up, status)
+            if self.out_f32 and not ops.can_use_few_rows(act, self.w_down):
+                return ops.linear(act, self.w_down, out_dtype=torch.float32)
             return ops.linear_few_rows(act, self.w_down, status)
         if self.interleave and h.shape[0] >= ops.TCGEN05_M_MIN and ops.can_use_tcgen05(h, self.w_gate_up):
             # many rows: the tcgen05 product with the SiLU gate in its epilogue (no activation pass over memory)
@@ -69,7 +71,38 @@ class GatedMLP(FeedForward):
             ops.silu_mul(gu, act, self.interleave)
         if ops.can_use_few_rows(act, self.w_down):
             return ops.linear_few_rows(act, self.w_down, status)
-        return ops.linear(act, self.w_down)
+        return ops.linear(act, self.w_down, out_dtype=torch.float32 if self.out_f32 else None)
+
+
+class GeluMLP(FeedForward):
+    """``down(gelu(up(h)))`` with the exact (erf) GELU, no gate, no biases.  Many rows in bfloat16: the GELU is the
+    epilogue of the tcgen05 up product; few rows: the K-split product's float32 slices go through one activation kernel;
+    float32: the activation kernel behind the float32 product.  The update leaves as float32 rows or slices."""
+
+    def __init__(self, width: int, inner: int, up_name: str, down_name: str):
+        self.width, self.inner = width, inner
+        self.names = (up_name, down_name)
+
+    def weight_specs(self):
+        u, d = self.names
+        return (WeightSpec(u, (self.inner, self.width)), WeightSpec(d, (self.width, self.inner)))
+
+    def bind(self, weights, rt) -> None:
+        u, d = self.names
+        self.w_up = weights[u].contiguous()
+        self.w_down = weights[d].contiguous()
+
+    def forward(self, ctx, h):
+        status = ctx.status if ctx is not None else None
+        if h.shape[0] >= ops.TCGEN05_M_MIN and ops.can_use_tcgen05(h, self.w_up):
+            if status is None:
+                status = torch.zeros(1, dtype=torch.int32, device=h.device)
+            act = ops.gemm_tcgen05(h, self.w_up, status, gelu=True)
+        else:
+            z = ops.linear_out_f32(h, self.w_up, status)
+            act = torch.empty((h.shape[0], self.inner), dtype=h.dtype, device=h.device)
+            ops.gelu_rows(z, act)
+        return ops.linear_out_f32(act, self.w_down, status)
 
 
 class ClampedGLU(FeedForward):
@@ -156,6 +189,10 @@ class RoutedExperts(FeedForward):
     largest choice scores); the weights are the chosen experts' s over their sum, times ``scale``.
     ``expert="gelu"``: an expert is ``down(gelu(up h))`` with the exact GELU and no gate; ``expert_names(e)`` then gives
     (up, down).  ``out_dtype`` float32: the weighted sum leaves as float32 rows (for a norm that reads it).
+    ``scored`` with ``renormalize=False``: the chosen scores times ``scale`` as they are.
+
+    ``weigh_input`` (SiLU-gated experts): a choice's weight multiplies what goes INTO the expert, the output is the plain
+    sum of expert(w * h); the kernels apply w to the first product's sums.
 
     ``over_all`` = dict(scale): a third way of weighing: the choice is the plain one (largest logits), the weights are
     the chosen experts' shares of the softmax over ALL experts, times ``scale``, not renormalised.
@@ -173,7 +210,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, inner: int, n_experts: int, top: int, router_name: str, router_bias_name: str | None,
                  expert_names, shared: FeedForward | None = None, scored: dict | None = None, expert: str = "silu_gated",
                  out_dtype: torch.dtype | None = None, over_all: dict | None = None, clamp: tuple[float, float] | None = None,
-                 shared_gate_name: str | None = None):
+                 shared_gate_name: str | None = None, weigh_input: bool = False):
         """``expert_names(e)`` -> (gate, up, down) tensor names of expert e."""
         if not 0 < top <= n_experts:
             raise ValueError(f"top={top} of {n_experts} experts")
@@ -185,6 +222,9 @@ class RoutedExperts(FeedForward):
             raise ValueError("the weights come from the softmax over all experts or from sigmoid scores, not both")
         if shared_gate_name is not None and shared is None:
             raise ValueError("a gate on the shared expert needs a shared expert")
+        if weigh_input and expert != "silu_gated":
+            raise ValueError("weights on an expert's input: SiLU-gated experts only")
+        self.weigh_input = bool(weigh_input)
         self.over_all = over_all
         self.clamp = (float(clamp[0]), float(clamp[1])) if clamp is not None else None
         self.shared_gate_name = shared_gate_name
@@ -227,7 +267,8 @@ class RoutedExperts(FeedForward):
             c = self.scored.get("correction")
             self.route_args = dict(correction=weights[c].contiguous() if c is not None else None,
                                    groups=int(self.scored.get("groups", 1)), keep=int(self.scored.get("keep", 1)),
-                                   scale=float(self.scored.get("scale", 1.0)))
+                                   scale=float(self.scored.get("scale", 1.0)),
+                                   renormalize=bool(self.scored.get("renormalize", True)))
         # [E, 2 * inner, width]: each expert's gate rows, then its up rows ([E, inner, width]: the up rows of an
         # ungated expert);  [E, width, inner]
         self.w_gate_up = torch.stack([torch.cat([weights[n] for n in names[:-1]], dim=0) for names in self.expert_names]).contiguous()
@@ -269,18 +310,20 @@ class RoutedExperts(FeedForward):
             tile_group = torch.empty((n_tiles,), dtype=torch.int32, device=dev)
             ops.moe_order(top_idx, E, offsets, order, place_of, pad=tile, tile_group=tile_group, src_token=src_token)
             rows = torch.empty((n_tiles * tile, self.width), dtype=h.dtype, device=dev)
-            ops.moe_gather(h, src_token, rows)
+            scale = torch.empty((n_tiles * tile,), dtype=torch.float32, device=dev) if self.weigh_input else None
+            ops.moe_gather(h, src_token, rows, order if self.weigh_input else None, top_w if self.weigh_input else None, scale)
             status = ctx.status if ctx is not None else torch.zeros(1, dtype=torch.int32, device=dev)
             act = ops.gemm_tcgen05_grouped(rows, self.w_gate_up_tc, tile_group, status, gated=not self.gelu, gelu=self.gelu,
-                                           clamp=self.clamp)
+                                           clamp=self.clamp, row_scale=scale)
             y = ops.gemm_tcgen05_grouped(act, self.w_down, tile_group, status)
-            ops.moe_combine(y, place_of, top_w, shared, out, shared_gate)
+            ops.moe_combine(y, place_of, top_w, shared, out, shared_gate, weigh=not self.weigh_input)
             return out
         order = torch.empty((T * top,), dtype=torch.int32, device=dev)
         ops.moe_order(top_idx, E, offsets, order, place_of)
         act = torch.empty((T * top, self.inner), dtype=h.dtype, device=dev)
-        ops.moe_gemm(h, self.w_gate_up, act, offsets, order, top, gated=not self.gelu, gelu=self.gelu, clamp=self.clamp)
+        ops.moe_gemm(h, self.w_gate_up, act, offsets, order, top, gated=not self.gelu, gelu=self.gelu, clamp=self.clamp,
+                     pair_scale=top_w if self.weigh_input else None)
         y = torch.empty((T * top, self.width), dtype=torch.float32, device=dev)
         ops.moe_gemm(act, self.w_down, y, offsets, None, top, gated=False)
-        ops.moe_combine(y, place_of, top_w, shared, out, shared_gate)
+        ops.moe_combine(y, place_of, top_w, shared, out, shared_gate, weigh=not self.weigh_input)
         return out

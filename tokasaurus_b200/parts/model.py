@@ -45,8 +45,9 @@ class DecoderModel(Part):
         for c in self.run_order:
             if not c.write_cache and c.cache not in writers:
                 raise ValueError(f"a layer call reads cache entry {c.cache} that no call writes")
-        # state that a block's input stages keep per request: an entry of its own for every layer call and stage
-        # (a block named in two calls runs over two different streams), numbered behind the mixers' entries
+        # what a block holds beside its mixer's entry (state of its input stages, further entries of a mixer made of several):
+        # an entry of its own for every layer call and name (a block named in two calls runs over two different
+        # streams), numbered behind the mixers' entries
         nxt = max([c.cache for c in self.run_order], default=-1) + 1
         self.stage_entries: list[dict[str, int]] = []
         self._stage_needs: dict[int, object] = {}
@@ -97,7 +98,7 @@ class DecoderModel(Part):
         return out
 
     def mixers(self):
-        return [b.mixer for b in self.blocks]
+        return [m for b in self.blocks for m in (b.mixer.inner_mixers() if hasattr(b.mixer, "inner_mixers") else (b.mixer,))]
 
     def cache_entries(self):
         """{cache entry: the need of the mixer that uses it}."""
@@ -126,8 +127,5 @@ class DecoderModel(Part):
             else:
                 stream = self.blocks[call.block].forward(ctx, stream, cache, rows if i == last else None)
             if taps is not None:
-                x = stream.x.clone()
-                if stream.delta is not None:
-                    x += stream.delta.sum(0) if stream.delta.dim() == 3 else stream.delta
-                taps.append(x)
+                taps.append(stream.settled())
         return self.head.forward(ctx, stream)

@@ -11,7 +11,11 @@ from tokasaurus_b200.parts.base import Norm, ResidualStream, WeightSpec
 
 
 class RMSNorm(Norm):
-    def __init__(self, width: int, eps: float, weight_name: str):
+    """``around_zero``: the weight is stored around zero and counts as 1 + w.  ``gain``: a number that multiplies the
+    result (a head's factor on its logits, say); it rides in the float32 weight."""
+
+    def __init__(self, width: int, eps: float, weight_name: str, around_zero: bool = False, gain: float = 1.0):
+        self.around_zero, self.gain = bool(around_zero), float(gain)
         self.width = width
         self.eps = float(eps)
         self.weight_name = weight_name
@@ -22,7 +26,10 @@ class RMSNorm(Norm):
         return (WeightSpec(self.weight_name, (self.width,), role="vector"),)
 
     def bind(self, weights, rt) -> None:
-        self.weight = weights[self.weight_name]
+        w = weights[self.weight_name]
+        if self.around_zero or self.gain != 1.0:
+            w = ((w.double() + (1.0 if self.around_zero else 0.0)) * self.gain).float().contiguous()
+        self.weight = w
         self.out_dtype = rt.dtype
 
     def _run(self, x: torch.Tensor, delta=None) -> torch.Tensor:

@@ -263,6 +263,158 @@ class Retention(Mixer):
         return ops.linear_out_f32(o, self.w_o, ctx.status)
 
 
+class MatrixMemory(Mixer):
+    """A matrix memory with exponential gates (the matrix cell of xLSTM): per head, with a running maximum m (0 at
+    admission) that keeps the exponentials in range,
+
+        m_t = max(f_t + m_(t-1), i_t),    S_t = exp(f_t + m_(t-1) - m_t) S_(t-1) + exp(i_t - m_t) k_t v_t^T,
+        n_t the same with k_t alone,      o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + den_eps),
+
+    where q_t is scaled by ``q_scale`` (None: dim^(-1/2)) and the log gates are soft-capped:
+    i = cap tanh((W_i h + b_i) / cap), f = log_sigmoid(cap tanh((W_f h + b_f) / cap)).  Every head's o_t is divided by its
+    root mean square; all heads' values are multiplied by one weight vector and by sigmoid(W_g h), and projected.
+
+    What a request carries (float32, zero at admission): S^T and n of every head (n as one more column of S, whose values
+    are all 1) and m.  The walk over the tokens is the kernel of the other linear-attention mixers
+    (csrc/decay_recurrence.cu) with decays and key scales made from the gates beforehand."""
+
+    graph_safe = True
+
+    def __init__(self, width: int, n_heads: int, dim: int, vdim: int, gate_cap: float, norm_eps: float, den_eps: float,
+                 names: dict, q_scale: float | None = None):
+        """``names``: tensor names under q, k, v, g, o, norm, i, i_b, f, f_b."""
+        if not gate_cap > 0:
+            raise ValueError(f"the gates' cap must be positive, got {gate_cap}")
+        self.width, self.n_heads, self.dim, self.vdim = width, n_heads, dim, vdim
+        self.gate_cap, self.norm_eps, self.den_eps = float(gate_cap), float(norm_eps), float(den_eps)
+        self.q_scale = float(dim) ** -0.5 if q_scale is None else float(q_scale)
+        self.names = dict(names)
+        self.defines = ops.decay_recurrence_defines(dim, vdim)  # refuses sizes the kernel does not take
+        self.walk_builds = ops.decay_walk_modules(dim, vdim)
+        self.m_off = n_heads * (vdim + 1) * dim  # where the running maxima stand in a slot's state
+
+    def weight_specs(self):
+        n, H, d, e = self.names, self.n_heads, self.dim, self.vdim
+        return (WeightSpec(n["q"], (H * d, self.width)), WeightSpec(n["k"], (H * d, self.width)),
+                WeightSpec(n["v"], (H * e, self.width)), WeightSpec(n["g"], (H * e, self.width)),
+                WeightSpec(n["i"], (H, self.width)), WeightSpec(n["f"], (H, self.width)),
+                WeightSpec(n["i_b"], (H,), role="vector"), WeightSpec(n["f_b"], (H,), role="vector"),
+                WeightSpec(n["norm"], (H * e,), role="vector"), WeightSpec(n["o"], (self.width, H * e)))
+
+    def kernel_modules(self, dtype):
+        return tuple(("decay_recurrence.cu", d) for d in self.walk_builds)
+
+    def cache_need(self):
+        # [S^T and n of every head: heads x (vdim + 1) x dim | m: heads], in whole 16-byte pieces
+        return StateNeed((-(-(self.m_off + self.n_heads) // 4) * 4,), "float32")
+
+    def bind(self, weights, rt) -> None:
+        n = self.names
+        self.w_in = torch.cat([weights[n[k]] for k in ("q", "k", "v", "g", "i", "f")], dim=0).contiguous()
+        self.w_o = weights[n["o"]].contiguous()
+        self.i_b, self.f_b = weights[n["i_b"]].contiguous(), weights[n["f_b"]].contiguous()
+        self.norm_w = weights[n["norm"]].contiguous()
+
+    def in_matrix(self) -> torch.Tensor:
+        return self.w_in
+
+    def out_matrix(self) -> torch.Tensor:
+        return self.w_o
+
+    def drop_matrices(self) -> None:
+        """The matrices live on in a wider product."""
+        self.w_in = self.w_o = None
+
+    def out_columns(self) -> int:
+        return self.n_heads * self.vdim
+
+    def mix(self, ctx, proj, cache, dtype, out_rows=None, out=None, out_scale: float = 1.0):
+        """From the float32 product ``proj`` [T, q | k | v | g | i | f] (a column slice will do) to what the output product
+        reads, times ``out_scale``, in ``dtype``; ``out``: where it goes, a column slice of a wider tensor."""
+        H, d, e = self.n_heads, self.dim, self.vdim
+        T, dev = proj.shape[0], proj.device
+        q, k = proj[:, :H * d], proj[:, H * d:2 * H * d]
+        v, g_off = proj[:, 2 * H * d:2 * H * d + H * e], 2 * H * d + H * e
+        i_off = g_off + H * e
+        dt_dec = torch.empty((T, 2 * H), dtype=torch.float32, device=dev)
+        floor = torch.empty((T, H), dtype=torch.float32, device=dev)
+        ops.memory_gates(proj, i_off, i_off + H, self.i_b, self.f_b, self.gate_cap, cache.state, self.m_off, ctx.seq_slot,
+                         ctx.seq_q_start, ctx.seq_q_len, ctx.n_seqs, dt_dec, floor, self.defines, cache.writable)
+        raw = torch.empty((T, H * e), dtype=torch.float32, device=dev)
+        den = torch.empty((T, H), dtype=torch.float32, device=dev)
+        ops.decay_walk(q, k, v, 1, dt_dec, None, None, cache.state, raw, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
+                       ctx.n_seqs, H, d, e, cache.writable, ones_out=den)
+        if out is None:
+            out = torch.empty((T, H * e), dtype=dtype, device=dev)
+        ops.memory_norm(raw, den, floor, proj, g_off, self.norm_w, self.q_scale, self.den_eps, self.norm_eps, out_scale, out,
+                        H, e, self.defines)
+        return out if out_rows is None else _rows(out, out_rows)
+
+    def forward(self, ctx, h, cache, out_rows=None):
+        proj = ops.linear(h, self.w_in, out_dtype=torch.float32)
+        return ops.linear_out_f32(self.mix(ctx, proj, cache, h.dtype, out_rows), self.w_o, ctx.status)
+
+
+class RealGatedRecurrence(Mixer):
+    """Griffin's recurrent block with a real-gated linear recurrent unit, a state of one number a channel:
+
+        y = gelu_tanh(W_y h + b_y),   u = conv(W_x h + b_x)  (a causal convolution a channel with a bias),
+        r, i = sigmoid of u through block-diagonal matrices,   log a = -decay_scale * r * softplus(lam),
+        S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t,   output W_o (S y).
+
+    A request carries S and the convolution's last ``taps - 1`` inputs (float32, zero at admission) in its slot.  The two
+    input projections are one product with a float32 result; convolution, gates, decays and recurrence are float32
+    (csrc/gated_recurrence.cu)."""
+
+    graph_safe = True
+
+    def __init__(self, width: int, inner: int, blocks: int, taps: int, decay_scale: float, names: dict):
+        """``inner``: channels of both branches, in ``blocks`` equal parts.  ``names``: tensor names under y, y_b, x, x_b,
+        conv, conv_b, ra, ra_b, ri, ri_b, lam, o."""
+        if blocks <= 0 or inner % blocks:
+            raise ValueError(f"{inner} channels do not divide into {blocks} equal parts")
+        if taps < 1:
+            raise ValueError(f"a convolution needs at least one tap, got {taps}")
+        self.width, self.inner, self.blocks, self.taps = width, inner, blocks, int(taps)
+        self.decay_scale, self.names = float(decay_scale), dict(names)
+
+    def weight_specs(self):
+        n, C, B, W = self.names, self.inner, self.blocks, self.width
+        part = C // B
+        return (WeightSpec(n["y"], (C, W)), WeightSpec(n["x"], (C, W)), WeightSpec(n["o"], (W, C)),
+                WeightSpec(n["ra"], (B, part, part)), WeightSpec(n["ri"], (B, part, part)),
+                WeightSpec(n["y_b"], (C,), role="vector"), WeightSpec(n["x_b"], (C,), role="vector"),
+                WeightSpec(n["conv"], (C, self.taps), role="vector"), WeightSpec(n["conv_b"], (C,), role="vector"),
+                WeightSpec(n["ra_b"], (B, part), role="vector"), WeightSpec(n["ri_b"], (B, part), role="vector"),
+                WeightSpec(n["lam"], (C,), role="vector"))
+
+    def kernel_modules(self, dtype):
+        return (("gated_recurrence.cu", None),)
+
+    def cache_need(self):
+        # [S: channels | the convolution's last taps - 1 inputs: (taps - 1) x channels]
+        return StateNeed((self.inner * self.taps,), "float32")
+
+    def bind(self, weights, rt) -> None:
+        n = self.names
+        self.w_in = torch.cat([weights[n["y"]], weights[n["x"]]], dim=0).contiguous()
+        self.w_o = weights[n["o"]].contiguous()
+        for k in ("ra", "ri", "y_b", "x_b", "conv", "conv_b"):
+            setattr(self, k, weights[n[k]].contiguous())
+        self.ra_b, self.ri_b = weights[n["ra_b"]].reshape(-1).contiguous(), weights[n["ri_b"]].reshape(-1).contiguous()
+        self.neg = (-self.decay_scale * torch.nn.functional.softplus(weights[n["lam"]].double())).float().contiguous()
+
+    def forward(self, ctx, h, cache, out_rows=None):
+        proj = ops.linear(h, self.w_in, out_dtype=torch.float32)
+        out = torch.empty((h.shape[0], self.inner), dtype=h.dtype, device=h.device)
+        ops.real_gated_recurrence(proj, 0, self.inner, self.y_b, self.x_b, self.conv, self.conv_b, self.ra, self.ra_b, self.ri,
+                                  self.ri_b, self.neg, cache.state, ctx.token_seq, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
+                                  out, cache.writable)
+        if out_rows is not None:
+            out = _rows(out, out_rows)
+        return ops.linear_out_f32(out, self.w_o, ctx.status)
+
+
 def _rows(t: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
     cut = torch.empty((rows.numel(), t.shape[1]), dtype=t.dtype, device=t.device)
     ops.gather_rows(t, rows, cut)

@@ -29,6 +29,13 @@ softmax of its own over the same values; the cached row is [k of map 0 | k of ma
 maps' outputs is a subclass's business (``_combine``; ``parts.diff_attention.DifferentialAttention``).  ``extra_names``:
 further matrices over the mixer's input whose rows ride in the same product as q, k and v (an output gate's, say);
 their float32 results are the trailing columns of the product that ``_combine`` is handed.
+
+``chunk``: instead of a sliding window, the sequence is cut into chunks of so many positions, counted from position 0,
+and a query sees the keys of its own chunk only; pages of earlier chunks go back.  ``distance_bias``: a number a head;
+that slope times the distance i - j comes off the scores, after scale and cap.
+
+A mixer that stands beside others reads a share of ONE input product and leaves its rows for ONE output product:
+``in_matrix`` / ``out_matrix`` are the matrices it wants there, ``mix`` is what lies between them.
 """
 
 from __future__ import annotations
@@ -48,7 +55,8 @@ class SinkAttention(Mixer):
                  out_bias_name: str | None = None, unit_norm: bool = True, qk_norm_names: tuple[str, str] | None = None,
                  rotary=None, rotary_pairs: bool = True, values_are_keys: bool = False,
                  head_scale_name: str | None = None, head_bias_name: str | None = None, weights: str = "softmax",
-                 keep_first: int = 0, maps: int = 1, extra_names: tuple[tuple[str, int], ...] = ()):
+                 keep_first: int = 0, maps: int = 1, extra_names: tuple[tuple[str, int], ...] = (),
+                 chunk: int | None = None, distance_bias=None):
         """``extra_names``: (tensor name, rows) of matrices [rows, width] appended to the q|k|v product."""
         if n_heads % n_kv_heads:
             raise ValueError(f"n_heads={n_heads} is not a multiple of n_kv_heads={n_kv_heads}")
@@ -64,6 +72,13 @@ class SinkAttention(Mixer):
             raise ValueError("several attention maps a head need a part that combines them, and values of their own")
         if keep_first < 0 or (keep_first and not window):
             raise ValueError("positions kept in sight need a window to be kept from")
+        if chunk and window:
+            raise ValueError("a chunk or a sliding window, not both")
+        if distance_bias is not None and (len(distance_bias) != n_heads or maps != 1):
+            raise ValueError(f"{len(distance_bias)} distance slopes for {n_heads} heads of {maps} maps")
+        self.chunk = int(chunk) if chunk else None
+        self.distance_bias = tuple(float(x) for x in distance_bias) if distance_bias is not None else None
+        self.head_slope: torch.Tensor | None = None
         self.maps, self.keep_first, self.extra_names = int(maps), int(keep_first), tuple(extra_names)
         if rotary is not None and rotary.rotary_dim > dim:
             raise ValueError(f"{rotary.rotary_dim} rotated channels in heads of {dim}")
@@ -79,7 +94,7 @@ class SinkAttention(Mixer):
         self.norm_eps, self.unit_norm = float(norm_eps), bool(unit_norm)
         self.names = (q_name, k_name, v_name, o_name)
         self.sink_name, self.bias_names, self.out_bias_name = sink_name, bias_names, out_bias_name
-        self.defines = ops.sink_attention_defines(dim, vdim, self.sigmoid, self.maps)
+        self.defines = ops.sink_attention_defines(dim, vdim, self.sigmoid, self.maps, self.distance_bias is not None)
         self.sinks = self.qkv_bias = self.out_bias = None
 
     def weight_specs(self):
@@ -106,8 +121,8 @@ class SinkAttention(Mixer):
         return (("attention_sink.cu", self.defines),)
 
     def cache_need(self):
-        return PagedCacheNeed(self.n_kv_heads, self.maps * self.dim + self.vdim, self.window, planes=1,
-                              keep_first=self.keep_first)
+        return PagedCacheNeed(self.n_kv_heads, self.maps * self.dim + self.vdim, self.chunk or self.window, planes=1,
+                              keep_first=self.keep_first, chunked=self.chunk is not None)
 
     def bind(self, weights, rt) -> None:
         q, k, v, o = self.names
@@ -123,6 +138,8 @@ class SinkAttention(Mixer):
             self.qk_norm_w = torch.stack([weights[n].float() for n in self.qk_norm_names]).contiguous()
         if self.rotary is not None and self.rotary.rotary_dim > 0:
             self.rot_freq = self.rotary.inv_freq64().to(rt.device)
+        if self.distance_bias is not None:
+            self.head_slope = torch.tensor(self.distance_bias, dtype=torch.float64).float().to(rt.device)
         if self.head_scale_name is not None:
             self.head_scale = weights[self.head_scale_name].contiguous()
         if self.head_bias_name is not None:
@@ -138,35 +155,53 @@ class SinkAttention(Mixer):
         rows (None: all)."""
         return attn
 
+    def in_matrix(self) -> torch.Tensor:
+        return self.w_qkv
+
+    def out_matrix(self) -> torch.Tensor:
+        return self.w_o
+
+    def drop_matrices(self) -> None:
+        """The matrices live on in a wider product."""
+        self.w_qkv = self.w_o = None
+
+    def out_columns(self) -> int:
+        return self.n_heads * self.vdim
+
     def forward(self, ctx, h, cache, out_rows=None):
-        H, G, d, e, M = self.n_heads, self.n_kv_heads, self.dim, self.vdim, self.maps
-        T = h.shape[0]
-        tables = ctx.tables[cache.group]
         qkv = ops.linear(h, self.w_qkv, out_dtype=torch.float32)
-        q = torch.empty((T, H * M * d), dtype=h.dtype, device=h.device)
+        return ops.linear_out_f32(self.mix(ctx, qkv, cache, h.dtype, out_rows), self.w_o, ctx.status)
+
+    def mix(self, ctx, qkv, cache, dtype, out_rows=None, out=None, out_scale: float = 1.0):
+        """From the float32 product ``qkv`` of all tokens (a column slice will do) to what the output product reads, times
+        ``out_scale``, in ``dtype``.  ``out`` (one map, all rows): where it goes, a column slice of a wider tensor."""
+        H, G, d, e, M = self.n_heads, self.n_kv_heads, self.dim, self.vdim, self.maps
+        T, dev = qkv.shape[0], qkv.device
+        tables = ctx.tables[cache.group]
+        q = torch.empty((T, H * M * d), dtype=dtype, device=dev)
         ops.sink_attn_prep(qkv, self.qkv_bias, self.unit_norm, self.norm_eps, q, cache.k, ctx.positions, ctx.token_seq,
                            tables.indptr, tables.page_ids, H, G, d, e, cache.page_size, cache.writable, ctx.status,
                            norm_w=self.qk_norm_w, rot_freq=self.rot_freq,
                            rot_dims=self.rotary.rotary_dim if self.rot_freq is not None else 0,
-                           rot_pairs=self.rotary_pairs, values_are_keys=self.values_are_keys, sigmoid=self.sigmoid, maps=M)
-        out_dtype = h.dtype if M == 1 else torch.float32  # several maps' outputs stay unrounded for what combines them
-        if ops.can_use_attn_sink_tc(h.dtype, d, e, M):
+                           rot_pairs=self.rotary_pairs, values_are_keys=self.values_are_keys, sigmoid=self.sigmoid, maps=M,
+                           distance=self.head_slope is not None)
+        out_dtype = dtype if M == 1 else torch.float32  # several maps' outputs stay unrounded for what combines them
+        options = dict(head_scale=self.head_scale, head_bias=self.head_bias, sigmoid=self.sigmoid, maps=M,
+                       keep_first=self.keep_first, chunk=self.chunk, head_slope=self.head_slope, out_scale=out_scale)
+        if ops.can_use_attn_sink_tc(dtype, d, e, M):
             # bfloat16: every token on the tensor cores (single tokens and portions by a kernel each); wanted rows are
             # cut out afterwards
-            attn = torch.empty((T, H * M * e), dtype=out_dtype, device=h.device)
+            attn = out if out is not None else torch.empty((T, H * M * e), dtype=out_dtype, device=dev)
             ops.attn_sink_tc(q, attn, cache.k, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, tables.indptr,
                              tables.page_ids, ctx.n_seqs, self.sinks, H, G, d, e, cache.page_size, self.scale, self.softcap,
-                             self.window, ctx.status, portions=not ctx.single_token_step, head_scale=self.head_scale,
-                             head_bias=self.head_bias, sigmoid=self.sigmoid, maps=M, keep_first=self.keep_first)
+                             self.window, ctx.status, portions=not ctx.single_token_step, **options)
             if out_rows is not None:
-                cut = torch.empty((out_rows.numel(), H * M * e), dtype=out_dtype, device=h.device)
+                cut = torch.empty((out_rows.numel(), H * M * e), dtype=out_dtype, device=dev)
                 ops.gather_rows(attn, out_rows, cut)
                 attn = cut
-            return ops.linear_out_f32(self._combine(ctx, attn, qkv, out_rows), self.w_o, ctx.status)
+            return self._combine(ctx, attn, qkv, out_rows)
         n_rows = T if out_rows is None else out_rows.numel()
-        attn = torch.empty((n_rows, H * M * e), dtype=out_dtype, device=h.device)
+        attn = out if out is not None else torch.empty((n_rows, H * M * e), dtype=out_dtype, device=dev)
         ops.attn_sink(q, attn, cache.k, ctx.token_seq, ctx.positions, tables.indptr, tables.page_ids, out_rows, n_rows,
-                      self.sinks, H, G, d, e, cache.page_size, self.scale, self.softcap, self.window, ctx.status,
-                      head_scale=self.head_scale, head_bias=self.head_bias, sigmoid=self.sigmoid, maps=M,
-                      keep_first=self.keep_first)
-        return ops.linear_out_f32(self._combine(ctx, attn, qkv, out_rows), self.w_o, ctx.status)
+                      self.sinks, H, G, d, e, cache.page_size, self.scale, self.softcap, self.window, ctx.status, **options)
+        return self._combine(ctx, attn, qkv, out_rows)
