@@ -8,6 +8,8 @@
 // What a request carries in its slot: S [C] and the convolution's last K - 1 inputs [K - 1, C], float32.  Everything here
 // is float32: the projections [y | x] arrive as float32 rows of one product, u, gates, decays and the recurrence stay
 // float32; only out leaves in the activation type.  sqrt(1 - a^2) is sqrt(-expm1(2 log a)), exact where a is close to 1.
+// A decay close to 1 is kept as a - 1 = expm1(log a) and applied as S + ((a - 1) S + x): rounding a itself would be the
+// same error at every token of a long memory, and those add up.
 //
 // The recurrence over a step's tokens is a scan in two kernels over tiles of MT consecutive tokens of the step, whatever
 // requests they belong to (a request's first token of the step starts from its slot's S and forgets what came before
@@ -131,7 +133,13 @@ __device__ __forceinline__ void convolve(const Conv& cv, const Step& st, const f
   }
 }
 
-// The scan within a tile.  sa, sx [MT][NT + 1]: decays and inputs; afterwards P and Sl go to memory.  Threads: NT
+// A decay as one number d: a - 1 (not positive) for decays above a half, else a itself (positive, however small).
+__device__ __forceinline__ float decay_code(float log_a) {
+  return log_a > -0.6931471f ? expm1f(log_a) : fmaxf(expf(log_a), 1e-37f);
+}
+__device__ __forceinline__ float decayed(float d, float S, float x) { return d <= 0.f ? S + fmaf(d, S, x) : fmaf(d, S, x); }
+
+// The scan within a tile.  sa, sx [MT][NT + 1]: decays (coded) and inputs; afterwards P and Sl go to memory.  Threads: NT
 // channels times SEGS runs of MT / SEGS tokens.
 template <int MT, int NT, int SEGS>
 __device__ __forceinline__ void tile_scan(float* sa, float* sx, float* ends, const Step& st, const float* __restrict__ state,
@@ -150,11 +158,11 @@ __device__ __forceinline__ void tile_scan(float* sa, float* sx, float* ends, con
       } else {
         const float a = sa[r * LD + ch], x = sx[r * LD + ch];
         if (s_idx[r] == 0) {  // the request's first token of this step starts from its slot
-          S = fmaf(a, state[(size_t)st.seq_slot[s_seq[r]] * slot_stride + c], x);
+          S = decayed(a, state[(size_t)st.seq_slot[s_seq[r]] * slot_stride + c], x);
           P = 0.f;
         } else {
-          S = fmaf(a, S, x);
-          P *= a;
+          S = decayed(a, S, x);
+          P = decayed(a, P, 0.f);
         }
       }
       sx[r * LD + ch] = S;
@@ -182,7 +190,7 @@ __device__ __forceinline__ void tile_scan(float* sa, float* sx, float* ends, con
 
 __device__ __forceinline__ void decay_and_input(float r_pre, float i_pre, float u, float neg, float& a, float& x) {
   const float log_a = neg * sigmoid_f(r_pre);
-  a = expf(log_a);
+  a = decay_code(log_a);
   x = sqrtf(-expm1f(2.f * log_a)) * sigmoid_f(i_pre) * u;
 }
 
