@@ -2,7 +2,7 @@
 random weights (the metric and configuration of BASELINE.json's configs[2]).
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 2|3|4]
-    python bench.py --design sozurax|daborax|verozen|bibalix   (another workload, see run_design; the default workload and its output line are unchanged)
+    python bench.py --design sozurax|daborax|verozen|bibalix|safupel   (another workload, see run_design; the default workload and its output line are unchanged)
 
 Prints ONE JSON line.  ``value``: decoded tokens a second at batch 8, each request holding a
 2,048-token prompt in the cache, timed on the device with CUDA events around K decode steps
@@ -160,7 +160,7 @@ def prefill_flops(m: dict, T: int, rows: int = 1) -> float:
     return linear + attention
 
 
-TIMED_OPS = ("diff_combine", "head_sigmoid_gate", "moe_logits", "sum_group_norm", "gelu_gate_rows", "gla_gates", "rotate_scale", "linear_out_f32", "scaled_norm_add", "cast_rows", "add_sinusoid", "clamped_glu", "gated_group_norm", "ssm_prep", "decay_walk",
+TIMED_OPS = ("real_gated_recurrence", "memory_gates", "memory_norm", "gelu_rows", "diff_combine", "head_sigmoid_gate", "moe_logits", "sum_group_norm", "gelu_gate_rows", "gla_gates", "rotate_scale", "linear_out_f32", "scaled_norm_add", "cast_rows", "add_sinusoid", "clamped_glu", "gated_group_norm", "ssm_prep", "decay_walk",
              "sink_attn_prep", "attn_sink", "attn_sink_tc", "silu_cols", "gemm_tcgen05_clamped", "add_layernorm", "add_layernorm_conv1", "short_conv", "polynorm", "gated_recurrence", "latent_prep",
              "rotate_pairs", "latent_attn", "moe_route", "moe_order", "moe_gather", "moe_gemm", "moe_combine",
              "gemm_tcgen05_grouped", "embed_gather", "add_rmsnorm", "rope_kv_write", "rope_kv_write_partials", "linear_decode", "linear_smallm",
@@ -734,6 +734,28 @@ def bibalix_configs(name: str) -> dict:
     return dict(bibalix=bib, sozurax=soz)
 
 
+def safupel_configs(name: str) -> dict:
+    """Layer sizes for ``--design safupel``: two sizes that resemble a real model's layers, each as a Safupel decoder
+    (a real-gated recurrence with a dense feed-forward, chunked attention beside a matrix memory with routed experts, the
+    recurrence again with a dense feed-forward and with routed experts; sublayers side by side under one norm) and as the
+    closest existing model, the Daborax decoder of ``daborax_configs`` (a walk over a matrix state, a convolution with a
+    recurrence behind it, windowed attention of the same kernel file, RMS norms, a dense feed-forward of the same inner
+    size) at the same width, depth, vocabulary and head sizes; the like of its routed experts is the Verozen decoder's."""
+    sizes = dict(w2048=dict(width=2048, heads=16, ff=8192, att_heads=16, att_kv=4, blocks=8, experts=16, top=4, expert_ff=2048, shared_ff=2048),
+                 w4096=dict(width=4096, heads=32, ff=14336, att_heads=32, att_kv=8, blocks=16, experts=16, top=4, expert_ff=3584, shared_ff=3584))
+    z = sizes[name]
+    W = z["width"]
+    dense = dict(kind="dense", ff=z["ff"])
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"]), router=dict(experts=z["experts"], top=z["top"]), shared=dict(ff=z["shared_ff"]))
+    rec = dict(type="rglru", mixer=dict(width=W, blocks=z["blocks"], conv=4))
+    par = dict(type="parallel", mixer=dict(
+        left=dict(heads=z["att_heads"], kv_heads=z["att_kv"], dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024)),
+        right=dict(heads=z["heads"], dim=128, vdim=128, gate_cap=15.0), left_scale=0.7, right_scale=0.7))
+    saf = dict(architecture="Safupel", vocab=32000, width=W, norm=dict(eps=1e-6), logit_scale=1.0,
+               layers=[dict(rec, mlp=dense), dict(par, mlp=moe), dict(rec, mlp=dense), dict(rec, mlp=moe)])
+    return dict(safupel=saf, daborax=daborax_configs(name)["daborax"], verozen=verozen_configs(name)["verozen"])
+
+
 def design_configs(name: str) -> dict:
     """Layer sizes for ``--design sozurax``: two sizes that resemble a real model's layers, each as a Sozurax decoder
     (a recurrent layer with a dense feed-forward, a latent-attention layer with routed experts, a second recurrent
@@ -763,7 +785,7 @@ def design_configs(name: str) -> dict:
 
 
 def run_design(args) -> dict:
-    """``--design sozurax|daborax|verozen|bibalix``: prefill (one 2,048-token prompt in one step) and decode (batch 8 and 64, prompts of
+    """``--design sozurax|daborax|verozen|bibalix|safupel``: prefill (one 2,048-token prompt in one step) and decode (batch 8 and 64, prompts of
     2,048 tokens in the cache) of that decoder at two layer sizes beside the closest existing decoder of equal size, random weights,
     bfloat16, with the CUDA-event time of each kind of kernel in one prefill step and one decode step of both."""
     import numpy as np
@@ -778,7 +800,7 @@ def run_design(args) -> dict:
     prompt_len, page_size = 2048, 16
     out = dict(design=args.design, dtype="bf16", data="synthetic", peaks=dict(peaks, source=peak_src), sizes={})
     configs_of = dict(daborax=daborax_configs, sozurax=design_configs, verozen=verozen_configs,
-                      bibalix=bibalix_configs)[args.design]
+                      bibalix=bibalix_configs, safupel=safupel_configs)[args.design]
     for size in ("w2048", "w4096"):
         res = {}
         for arch, cfg in configs_of(size).items():
@@ -891,7 +913,7 @@ def main() -> int:
     ap.add_argument("--config", type=int, default=2, choices=[2, 3, 4],
                     help="2: the headline metric (default); 3 and 4: the further workloads, see run_further")
     ap.add_argument("--design-arch", default=None, help="with --design: only this arm (the design's name or 'llama')")
-    ap.add_argument("--design", default=None, choices=["sozurax", "daborax", "verozen", "bibalix"],
+    ap.add_argument("--design", default=None, choices=["sozurax", "daborax", "verozen", "bibalix", "safupel"],
                     help="instead of the headline workload: this design's prefill and decode at two layer sizes beside "
                          "the closest existing decoder of equal size (see run_design)")
     args = ap.parse_args()

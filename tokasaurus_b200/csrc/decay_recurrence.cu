@@ -577,7 +577,7 @@ namespace {
 // a_t = exp(f_t + m_(t-1) - m_t), the key scale c_t = exp(i_t - m_t) and the floor exp(-m_t) of the denominator.  The
 // maximum is a scan of the pairs (f, i) under (f1, i1) then (f2, i2) = (f1 + f2, max(i1 + f2, i2)), a block's threads at
 // a time.  (The state's scale is exp(-m) whatever m is, so a rounding of m moves a, c and the floor together.)
-constexpr int GATE_THREADS = 128;
+constexpr int GATE_THREADS = 512;  // for portions; a step of single tokens takes one warp a (request, head)
 
 __global__ void __launch_bounds__(GATE_THREADS)
 memory_gates_kernel(const float* __restrict__ z, int stride, int i_off, int f_off, const float* __restrict__ i_bias,
@@ -597,7 +597,7 @@ memory_gates_kernel(const float* __restrict__ z, int stride, int i_off, int f_of
   float* mp = state + (size_t)seq_slot[s] * slot_stride + m_off + h;
   float m0 = *mp;  // the maximum before this round of tokens
   const float bi = i_bias[h], bf = f_bias[h], inv_cap = 1.f / cap;
-  for (int t0 = 0; t0 < n; t0 += GATE_THREADS) {
+  for (int t0 = 0; t0 < n; t0 += blockDim.x) {
     const int t = t0 + tid;
     const bool live = t < n;
     float gi = 0.f, gf = 0.f;
@@ -634,7 +634,7 @@ memory_gates_kernel(const float* __restrict__ z, int stride, int i_off, int f_of
       dt_dec[at * 2 * heads + heads + h] = expf(gf + (m_prev - m_t));
       floor_out[at * heads + h] = expf(-m_t);
     }
-    if (t == min(n, t0 + GATE_THREADS) - 1) m_last = m_t;
+    if (t == min(n, t0 + (int)blockDim.x) - 1) m_last = m_t;
     __syncthreads();
     m0 = m_last;  // (written again only after the next round's first barrier)
   }
@@ -643,8 +643,18 @@ memory_gates_kernel(const float* __restrict__ z, int stride, int i_off, int f_of
 
 // out[t][head's vdim values] = N(o) * w * sigmoid(g) * out_scale with o = S^T q / (max(|n . q|, floor) + den_eps), q scaled
 // by q_scale on the way, N the division by the head's root mean square.  raw float32 [T, heads * vdim], den and floor
-// float32 [T, heads], g float32 at column g_off of rows of g_stride.  One warp a (token, head).
-template <typename T>
+// float32 [T, heads], g float32 at column g_off of rows of g_stride.  One warp a (token, head); VEC: four values a lane and
+// step (vdim and all rows in whole 16-byte pieces), those of the first two steps kept for the second pass.
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<uint32_t*>(&a);
+  u.y = *reinterpret_cast<uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 memory_norm_kernel(const float* __restrict__ raw, const float* __restrict__ den, const float* __restrict__ floor_in,
                    const float* __restrict__ g, int g_stride, int g_off, const float* __restrict__ w, float q_scale,
@@ -657,19 +667,57 @@ memory_norm_kernel(const float* __restrict__ raw, const float* __restrict__ den,
   if (pair >= pairs) return;
   const long long t = pair / heads;
   const int h = (int)(pair - t * heads);
-  const float f = q_scale / (fmaxf(fabsf(den[pair] * q_scale), floor_in[pair]) + den_eps);
   const float* o = raw + pair * vdim;
-  float ss = 0.f;
-  for (int j = lane; j < vdim; j += 32) {
-    const float v = o[j] * f;
-    ss = fmaf(v, v, ss);
-  }
-  ss = warp_sum(ss);
-  const float r = f * rsqrtf(ss / (float)vdim + eps) * out_scale;
   const float* gr = g + t * g_stride + g_off + (long long)h * vdim;
   const float* wr = w + (long long)h * vdim;
   T* dst = out + t * out_stride + (long long)h * vdim;
-  for (int j = lane; j < vdim; j += 32) dst[j] = from_float<T>(o[j] * r * wr[j] / (1.f + expf(-gr[j])));
+  const float d = den[pair], fl = floor_in[pair];
+  float ss = 0.f;
+  if constexpr (VEC) {
+    constexpr int KEEP = 2;
+    float4 ov[KEEP], gv[KEEP], wv[KEEP];
+#pragma unroll
+    for (int k = 0; k < KEEP; k++) {
+      const int j = (lane + 32 * k) * 4;
+      if (j < vdim) {
+        ov[k] = *reinterpret_cast<const float4*>(o + j);
+        gv[k] = *reinterpret_cast<const float4*>(gr + j);
+        wv[k] = *reinterpret_cast<const float4*>(wr + j);
+      }
+    }
+    const float f = q_scale / (fmaxf(fabsf(d * q_scale), fl) + den_eps);
+    auto sq = [&](const float4& v) {
+      const float a = v.x * f, b = v.y * f, c = v.z * f, e = v.w * f;
+      ss += (a * a + b * b) + (c * c + e * e);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; k++)
+      if ((lane + 32 * k) * 4 < vdim) sq(ov[k]);
+    for (int j = (lane + 32 * KEEP) * 4; j < vdim; j += 128) sq(*reinterpret_cast<const float4*>(o + j));
+    ss = warp_sum(ss);
+    const float r = f * rsqrtf(ss / (float)vdim + eps) * out_scale;
+    auto gated = [&](const float4& v, const float4& gg, const float4& ww) {
+      return make_float4(v.x * r * ww.x / (1.f + expf(-gg.x)), v.y * r * ww.y / (1.f + expf(-gg.y)),
+                         v.z * r * ww.z / (1.f + expf(-gg.z)), v.w * r * ww.w / (1.f + expf(-gg.w)));
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; k++) {
+      const int j = (lane + 32 * k) * 4;
+      if (j < vdim) put4(dst + j, gated(ov[k], gv[k], wv[k]));
+    }
+    for (int j = (lane + 32 * KEEP) * 4; j < vdim; j += 128)
+      put4(dst + j, gated(*reinterpret_cast<const float4*>(o + j), *reinterpret_cast<const float4*>(gr + j),
+                          *reinterpret_cast<const float4*>(wr + j)));
+  } else {
+    const float f = q_scale / (fmaxf(fabsf(d * q_scale), fl) + den_eps);
+    for (int j = lane; j < vdim; j += 32) {
+      const float v = o[j] * f;
+      ss = fmaf(v, v, ss);
+    }
+    ss = warp_sum(ss);
+    const float r = f * rsqrtf(ss / (float)vdim + eps) * out_scale;
+    for (int j = lane; j < vdim; j += 32) dst[j] = from_float<T>(o[j] * r * wr[j] / (1.f + expf(-gr[j])));
+  }
 }
 
 template <typename T>
@@ -681,7 +729,11 @@ int memory_norm_launch(const float* raw, const float* den, const float* floor_in
   const long long pairs = (long long)n_tokens * heads;
   const long long blocks = (pairs + 7) / 8;
   if (blocks > 0x7fffffffLL) return -3;
-  return launch_pdl(memory_norm_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, st, raw, den, floor_in, g, g_stride, g_off, w,
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool vec = vdim % 4 == 0 && g_stride % 4 == 0 && g_off % 4 == 0 && out_stride % 4 == 0 && al16(raw) && al16(g) &&
+                   al16(w) && al16(out);
+  auto kernel = vec ? memory_norm_kernel<T, true> : memory_norm_kernel<T, false>;
+  return launch_pdl(kernel, dim3((unsigned)blocks), dim3(256), 0, st, raw, den, floor_in, g, g_stride, g_off, w,
                     q_scale, den_eps, eps, out_scale, (T*)out, out_stride, heads, vdim, pairs);
 }
 
@@ -689,12 +741,12 @@ int memory_norm_launch(const float* raw, const float* den, const float* floor_in
 
 TKB_EXPORT int tkb_memory_gates(const float* z, int stride, int i_off, int f_off, const float* i_bias, const float* f_bias,
                                 float cap, float* state, long long slot_stride, long long m_off, const int* seq_slot,
-                                const int* seq_q_start, const int* seq_q_len, int n_seqs, int heads, float* dt_dec,
-                                float* floor_out, int write_state, void* st) {
+                                const int* seq_q_start, const int* seq_q_len, int n_seqs, int n_tokens, int heads,
+                                float* dt_dec, float* floor_out, int write_state, void* st) {
   if (n_seqs <= 0) return 0;
   if (heads <= 0 || !(cap > 0.f)) return -2;
   if (heads > 65535) return -3;
-  return launch_pdl(memory_gates_kernel, dim3(n_seqs, heads), dim3(GATE_THREADS), 0, (cudaStream_t)st, z, stride, i_off,
+  return launch_pdl(memory_gates_kernel, dim3(n_seqs, heads), dim3(n_tokens > n_seqs ? GATE_THREADS : 32), 0, (cudaStream_t)st, z, stride, i_off,
                     f_off, i_bias, f_bias, cap, state, slot_stride, m_off, seq_slot, seq_q_start, seq_q_len, heads, dt_dec,
                     floor_out, write_state);
 }

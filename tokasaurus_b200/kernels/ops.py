@@ -1405,7 +1405,8 @@ def memory_gates(proj: torch.Tensor, i_off: int, f_off: int, i_bias: torch.Tenso
     _check(_fn(_libs.get("decay_recurrence.cu", **defines), "tkb_memory_gates")(
         _ptr(proj), c_int(proj.stride(0)), c_int(i_off), c_int(f_off), _ptr(i_bias), _ptr(f_bias), c_float(cap), _ptr(state),
         ctypes.c_longlong(state.stride(0)), ctypes.c_longlong(m_off), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len),
-        c_int(n_seqs), c_int(heads), _ptr(dt_dec), _ptr(floor), c_int(1 if write_state else 0), _stream()), "memory_gates")
+        c_int(n_seqs), c_int(T), c_int(heads), _ptr(dt_dec), _ptr(floor), c_int(1 if write_state else 0), _stream()),
+        "memory_gates")
 
 
 def memory_norm(raw: torch.Tensor, den: torch.Tensor, floor: torch.Tensor, gate: torch.Tensor, g_off: int, weight: torch.Tensor,
