@@ -7,7 +7,7 @@
 //
 // What a request carries in its slot: S [C] and the convolution's last K - 1 inputs [K - 1, C], float32.  Everything here
 // is float32: the projections [y | x] arrive as float32 rows of one product, u, gates, decays and the recurrence stay
-// float32; only out leaves in the activation type.  sqrt(1 - a^2) is sqrt(-expm1(2 log a)), exact where a is close to 1.
+// float32; only out leaves in the activation type.  1 - a^2 is -(a - 1)(a + 1) with a - 1 = expm1(log a) where a is close to 1.
 // A decay close to 1 is kept as a - 1 = expm1(log a) and applied as S + ((a - 1) S + x): rounding a itself would be the
 // same error at every token of a long memory, and those add up.
 //

@@ -5,7 +5,7 @@
 Each mixer keeps its own cache entry (the left one's is the layer call's, the right one's an entry beside it), and
 neither projects for itself: ONE product makes all of what both read from h, ONE product takes what both leave, laid
 side by side in a row and already multiplied by its factor, through both output matrices.  A mixer that can stand here
-gives ``in_matrix`` / ``out_matrix`` / ``out_columns`` and ``mix(ctx, rows of its share of the input product, cache, dtype,
+gives ``in_matrix`` / ``out_matrix`` / ``drop_matrices`` and ``mix(ctx, rows of its share of the input product, cache, dtype,
 out=..., out_scale=...)``.
 """
 

@@ -325,9 +325,6 @@ class MatrixMemory(Mixer):
         """The matrices live on in a wider product."""
         self.w_in = self.w_o = None
 
-    def out_columns(self) -> int:
-        return self.n_heads * self.vdim
-
     def mix(self, ctx, proj, cache, dtype, out_rows=None, out=None, out_scale: float = 1.0):
         """From the float32 product ``proj`` [T, q | k | v | g | i | f] (a column slice will do) to what the output product
         reads, times ``out_scale``, in ``dtype``; ``out``: where it goes, a column slice of a wider tensor."""

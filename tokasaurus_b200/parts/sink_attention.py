@@ -165,9 +165,6 @@ class SinkAttention(Mixer):
         """The matrices live on in a wider product."""
         self.w_qkv = self.w_o = None
 
-    def out_columns(self) -> int:
-        return self.n_heads * self.vdim
-
     def forward(self, ctx, h, cache, out_rows=None):
         qkv = ops.linear(h, self.w_qkv, out_dtype=torch.float32)
         return ops.linear_out_f32(self.mix(ctx, qkv, cache, h.dtype, out_rows), self.w_o, ctx.status)
