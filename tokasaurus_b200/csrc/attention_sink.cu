@@ -51,9 +51,16 @@
 // A bias by distance, chosen at compile time (-DTKB_DIST=1): head_slope (float32 [heads]) times the distance i - j comes
 // off the score, after scale and cap.
 //
-// Outputs go to rows of out_stride values, multiplied by out_scale (a mixer beside another writes its share of a wider row).
+// Outputs go to rows of out_stride values, multiplied by out_scale (a mixer beside another writes its share of a wider row)
+// and, if there is a gate, by the sigmoid of the (token, head)'s gate logit.
 //
-// Compile with -DTKB_QK=<query/key size> -DTKB_VD=<value size> [-DTKB_SIGMOID=1] [-DTKB_MAPS=2] [-DTKB_DIST=1].
+// A norm over the whole projection: sink_attn_prep can divide all of q, and all of k, by ONE root mean square each.
+// A layer that reads another layer's rows has no keys and values of its own: sink_attn_prep then makes q alone.
+//
+// -DTKB_TAPS=<n>: the build with sink_attn_conv_prep, which puts a causal convolution of n taps a channel between the
+// projections and the norm and rotation (below).
+//
+// Compile with -DTKB_QK=<query/key size> -DTKB_VD=<value size> [-DTKB_SIGMOID=1] [-DTKB_MAPS=2] [-DTKB_DIST=1] [-DTKB_TAPS=n].
 #include "common.cuh"
 #include <float.h>
 #include <type_traits>
@@ -71,6 +78,10 @@ static_assert(TKB_QK >= 1 && TKB_QK <= 512 && TKB_VD >= 1 && TKB_VD <= 512, "hea
 #ifndef TKB_DIST
 #define TKB_DIST 0
 #endif
+#ifndef TKB_TAPS
+#define TKB_TAPS 0
+#endif
+static_assert(TKB_TAPS >= 0 && TKB_TAPS <= 16, "up to 16 taps");
 static_assert(TKB_MAPS >= 1 && TKB_MAPS <= 4, "one to four attention maps a head");
 
 using namespace tkb;
@@ -91,6 +102,11 @@ constexpr bool DIST = TKB_DIST != 0;
 __device__ __forceinline__ int first_key(int p, int window, int chunk) {
   const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
   return chunk > 0 ? max(lo, p - p % chunk) : lo;
+}
+
+// The output gate of (token row, head): the sigmoid of its logit, 1 without a gate.
+__device__ __forceinline__ float head_gate(const float* __restrict__ gate, int stride, int row, int h) {
+  return gate != nullptr ? 1.f / (1.f + expf(-gate[(size_t)row * stride + h])) : 1.f;
 }
 
 template <typename T>
@@ -127,15 +143,18 @@ __device__ __forceinline__ float dot_key(const T* __restrict__ k, const float* _
 }
 
 // qkv: float32 [T, stride] = [q (nh * QK) | k (nkv * QK) | v (nkv * VD)]  (no v if values_are_keys)
-// norm_w: float32 [2][QK] weights of the q heads' and the k heads' norm, or null; freq: float64 [rot_dims / 2] or null
+// norm: 0 none, 1 every q and k vector by its own root mean square, 2 all of q at once and all of k at once
+// norm_w: float32 weights of the norm or null: [2][QK], of the q vectors and the k vectors; with norm 2 one for every
+// column of q and k;  freq: float64 [rot_dims / 2] or null.  own_kv 0: the rows hold no k and no v, nothing is cached.
 template <typename T>
 __global__ void __launch_bounds__(256)
-sink_attn_prep_kernel(const float* __restrict__ qkv, int stride, const float* __restrict__ bias, int unit_norm,
+sink_attn_prep_kernel(const float* __restrict__ qkv, int stride, const float* __restrict__ bias, int norm,
                       float eps, T* __restrict__ q_out, T* __restrict__ cache, const int* __restrict__ positions,
                       const int* __restrict__ token_seq, const int* __restrict__ page_indptr,
                       const int* __restrict__ page_ids, int nh, int nkv, int page_size, int num_pages, int write_cache,
                       int* __restrict__ status, const float* __restrict__ norm_w, const double* __restrict__ freq,
-                      int rot_dims, int rot_pairs, int values_are_keys) {
+                      int rot_dims, int rot_pairs, int values_are_keys, int own_kv) {
+  __shared__ float red[33];
   __shared__ float rot_cs[QK];  // [rot_dims / 2] cosines, then as many sines
   trigger_dependents();
   grid_dependency_wait();
@@ -146,7 +165,7 @@ sink_attn_prep_kernel(const float* __restrict__ qkv, int stride, const float* __
   const float* row = qkv + (size_t)t * stride;
   const int p = positions[t];
   int page = -1;
-  if (write_cache) page = checked_page(page_ids[page_indptr[s] + p / page_size], num_pages, status);
+  if (write_cache && own_kv) page = checked_page(page_ids[page_indptr[s] + p / page_size], num_pages, status);
   const int slot = p % page_size;
   const int half = freq != nullptr ? rot_dims / 2 : 0;
   if (half > 0) {
@@ -159,22 +178,37 @@ sink_attn_prep_kernel(const float* __restrict__ qkv, int stride, const float* __
     __syncthreads();
   }
   // q vectors and k vectors (MAPS of each a head): one warp a vector
-  const int nhq = nh * MAPS, nkk = nkv * MAPS;
+  const int nhq = nh * MAPS, nkk = own_kv ? nkv * MAPS : 0;
+  float r_all[2] = {1.f, 1.f};
+  if (norm == 2) {
+    for (int part = 0; part < 2; part++) {
+      const int c0 = part ? nhq * QK : 0, n = (part ? nkk : nhq) * QK;
+      float ss = 0.f;
+      for (int c = c0 + threadIdx.x; c < c0 + n; c += blockDim.x) {
+        const float v = row[c] + (bias ? bias[c] : 0.f);
+        ss = fmaf(v, v, ss);
+      }
+      ss = block_sum(ss, red);
+      r_all[part] = rsqrtf(ss / (float)max(n, 1) + eps);
+    }
+  }
   for (int hh = warp; hh < nhq + nkk; hh += nwarps) {
     const int off = hh * QK;  // the k vectors follow the q vectors in the row
-    float ss = 0.f;
-    for (int d = lane; d < QK; d += 32) {
-      const float v = row[off + d] + (bias ? bias[off + d] : 0.f);
-      ss = fmaf(v, v, ss);
+    float r = r_all[hh < nhq ? 0 : 1];
+    if (norm == 1) {
+      float ss = 0.f;
+      for (int d = lane; d < QK; d += 32) {
+        const float v = row[off + d] + (bias ? bias[off + d] : 0.f);
+        ss = fmaf(v, v, ss);
+      }
+      r = rsqrtf(warp_sum(ss) / (float)QK + eps);
     }
-    ss = warp_sum(ss);
-    const float r = unit_norm ? rsqrtf(ss / (float)QK + eps) : 1.f;
     T* dst = nullptr;
     if (hh < nhq) dst = q_out + (size_t)t * nhq * QK + off;
     else if (page >= 0)
       dst = cache + (((size_t)page * nkv + (hh - nhq) / MAPS) * page_size + slot) * ROW + ((hh - nhq) % MAPS) * QK;
     if (dst != nullptr) {
-      const float* w = norm_w ? norm_w + (hh < nhq ? 0 : QK) : nullptr;
+      const float* w = norm_w ? norm_w + (norm == 2 ? off : (hh < nhq ? 0 : QK)) : nullptr;
       auto val = [&](int d) { return (row[off + d] + (bias ? bias[off + d] : 0.f)) * r * (w ? w[d] : 1.f); };
       for (int i = lane; i < half; i += 32) {
         const int a = rot_pairs ? 2 * i : i, b = rot_pairs ? 2 * i + 1 : i + half;
@@ -195,6 +229,223 @@ sink_attn_prep_kernel(const float* __restrict__ qkv, int stride, const float* __
   }
 }
 
+// A short causal convolution a channel between the projections and what sink_attn_prep does:
+//   y_t[c] = sum_j taps[c][j] * u_(t - TAPS + 1 + j)[c],   u the projected values (q, k and v columns alike), zeros before
+// the request's first token.  A request's last TAPS - 1 projected rows are its state, float32 [TAPS - 1][columns] in its
+// slot (zero at admission), oldest first.
+//
+// Block (x, y): `tb` consecutive tokens, and share y of the vectors (q heads, k heads, v heads); a warp takes a vector
+// through the block's tokens, every row it needs fetched once and before the first sum.  A tap that reaches behind the
+// portion's first token reads the state.  Requests that bring one token have their state moved on here (the lane that
+// read a column's old values writes the new ones); longer portions leave it to sink_conv_state, launched behind.
+#if TKB_TAPS > 0
+constexpr int TAPS = TKB_TAPS;
+constexpr int HALO = TAPS - 1;
+constexpr int CPL = ((QK > VD ? QK : VD) + 31) / 32;    // values of a vector a lane
+constexpr int TB = CPL <= 4 ? 8 : (CPL <= 8 ? 4 : 2);   // most tokens a block takes
+constexpr int CONV_WARPS = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(CONV_WARPS * 32)
+sink_attn_conv_prep_kernel(const float* __restrict__ qkv, int stride, const float* __restrict__ taps, float* state,
+                           long long slot_stride, int norm, float eps, T* __restrict__ q_out, T* __restrict__ cache,
+                           const int* __restrict__ positions, const int* __restrict__ token_seq,
+                           const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
+                           const int* __restrict__ seq_q_len, const int* __restrict__ page_indptr,
+                           const int* __restrict__ page_ids, int n_tokens, int nh, int nkv, int page_size, int num_pages,
+                           int write_cache, int write_state, int* __restrict__ status, const float* __restrict__ norm_w,
+                           const double* __restrict__ freq, int rot_dims, int rot_pairs, int own_kv, int tb) {
+  __shared__ float rot_cs[TB][QK];
+  __shared__ float vecs[CONV_WARPS][QK];
+  __shared__ int tok_seq[TB], tok_idx[TB], tok_len[TB], tok_slot[TB], tok_page[TB], tok_pos[TB];
+  trigger_dependents();
+  grid_dependency_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = blockIdx.x * tb;
+  if ((int)threadIdx.x < tb) {
+    const int j = threadIdx.x, t = t0 + j;
+    const int s = t < n_tokens ? token_seq[t] : -1;
+    tok_seq[j] = s;
+    tok_page[j] = -1;
+    if (s >= 0) {
+      tok_idx[j] = t - seq_q_start[s];
+      tok_len[j] = seq_q_len[s];
+      tok_slot[j] = seq_slot[s];
+      tok_pos[j] = positions[t];
+      if (write_cache && own_kv)
+        tok_page[j] = checked_page(page_ids[page_indptr[s] + tok_pos[j] / page_size], num_pages, status);
+    }
+  }
+  __syncthreads();
+  const int half = freq != nullptr ? rot_dims / 2 : 0;
+  for (int i = threadIdx.x; i < tb * half; i += blockDim.x) {
+    const int j = i / half, e = i - j * half;
+    if (tok_seq[j] >= 0) {
+      double sn, cs;
+      sincos((double)tok_pos[j] * freq[e], &sn, &cs);
+      rot_cs[j][e] = (float)cs;
+      rot_cs[j][half + e] = (float)sn;
+    }
+  }
+  __syncthreads();
+  const int nhq = nh * MAPS, nkk = own_kv ? nkv * MAPS : 0, n_vec = nhq + nkk + (own_kv ? nkv : 0);
+  const int columns = (nhq + nkk) * QK + (own_kv ? nkv * VD : 0);
+  for (int hh = blockIdx.y * CONV_WARPS + warp; hh < n_vec; hh += gridDim.y * CONV_WARPS) {
+    const bool is_v = hh >= nhq + nkk;
+    const int off = is_v ? (nhq + nkk) * QK + (hh - nhq - nkk) * VD : hh * QK;
+    const int n = is_v ? VD : QK;
+    // projected values: u[HALO + j] of the block's token j, u[0 .. HALO - 1] of the tokens before the first
+    float u[HALO + TB][CPL], w[TAPS][CPL];
+#pragma unroll
+    for (int e = 0; e < HALO + TB; e++) {
+      const int t = t0 - HALO + e;
+      // rows before the block's first token count only if they belong to that token's portion
+      const bool live = e < HALO ? (tok_seq[0] >= 0 && tok_idx[0] >= HALO - e) : (e - HALO < tb && t < n_tokens);
+#pragma unroll
+      for (int i = 0; i < CPL; i++) {
+        const int d = lane + 32 * i;
+        u[e][i] = live && d < n ? qkv[(size_t)t * stride + off + d] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < CPL; i++) {
+      const int d = lane + 32 * i;
+#pragma unroll
+      for (int k = 0; k < TAPS; k++) w[k][i] = d < n ? taps[(size_t)(off + d) * TAPS + k] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < TB; j++) {
+      if (j >= tb || tok_seq[j] < 0) continue;
+      const int idx = tok_idx[j];
+      float* st = state + (size_t)tok_slot[j] * slot_stride + off;  // (not read or written if HALO is 0)
+      float y[CPL], prev[HALO > 0 ? HALO : 1][CPL];  // prev[o - 1]: the value o tokens back
+#pragma unroll
+      for (int o = 1; o <= HALO; o++)
+#pragma unroll
+        for (int i = 0; i < CPL; i++) {
+          const int d = lane + 32 * i;
+          prev[o - 1][i] = idx >= o ? u[HALO + j - o][i] : (d < n ? st[(size_t)(HALO + idx - o) * columns + d] : 0.f);
+        }
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < CPL; i++) {
+        y[i] = 0.f;
+#pragma unroll
+        for (int o = HALO; o >= 1; o--) y[i] = fmaf(w[HALO - o][i], prev[o - 1][i], y[i]);
+        y[i] = fmaf(w[HALO][i], u[HALO + j][i], y[i]);
+        ss = fmaf(y[i], y[i], ss);
+      }
+      if (HALO > 0 && write_state && tok_len[j] == 1) {
+#pragma unroll
+        for (int i = 0; i < CPL; i++) {
+          const int d = lane + 32 * i;
+          if (d < n) {
+#pragma unroll
+            for (int r = 0; r + 1 < HALO; r++) st[(size_t)r * columns + d] = prev[HALO - 2 - r][i];
+            st[(size_t)(HALO - 1) * columns + d] = u[HALO + j][i];
+          }
+        }
+      }
+      T* dst = nullptr;
+      if (hh < nhq) {
+        dst = q_out + (size_t)(t0 + j) * nhq * QK + off;
+      } else if (tok_page[j] >= 0) {
+        const int g = is_v ? hh - nhq - nkk : (hh - nhq) / MAPS;
+        dst = cache + (((size_t)tok_page[j] * nkv + g) * page_size + tok_pos[j] % page_size) * ROW +
+              (is_v ? KW : ((hh - nhq) % MAPS) * QK);
+      }
+      const bool normed = norm == 1 && !is_v;
+      if (normed) {
+        const float r = rsqrtf(warp_sum(ss) / (float)QK + eps);
+        const float* nw = norm_w ? norm_w + (hh < nhq ? 0 : QK) : nullptr;
+#pragma unroll
+        for (int i = 0; i < CPL; i++) {
+          const int d = lane + 32 * i;
+          y[i] *= r * (nw && d < n ? nw[d] : 1.f);
+        }
+      }
+      if (dst == nullptr) continue;
+      if (half > 0 && !is_v) {
+        float* v = vecs[warp];
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < CPL; i++)
+          if (lane + 32 * i < QK) v[lane + 32 * i] = y[i];
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < CPL; i++) {
+          const int d = lane + 32 * i;
+          if (d < 2 * half) {
+            // this channel's partner in its pair, and which of the two it is
+            const int e = rot_pairs ? d >> 1 : (d < half ? d : d - half);
+            const bool second = rot_pairs ? (d & 1) != 0 : d >= half;
+            const float o = v[rot_pairs ? d ^ 1 : (second ? d - half : d + half)];
+            const float c = rot_cs[j][e], sn = rot_cs[j][half + e];
+            y[i] = second ? y[i] * c + o * sn : y[i] * c - o * sn;
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < CPL; i++) {
+        const int d = lane + 32 * i;
+        if (d < n) dst[d] = from_float<T>(y[i]);
+      }
+    }
+  }
+}
+
+// The state behind portions of several tokens: the last HALO projected rows, counting on from the old state where a
+// portion is shorter than that.  Grid (request row, column tile); a thread owns a column.
+__global__ void sink_conv_state_kernel(const float* __restrict__ qkv, int stride, float* state, long long slot_stride,
+                                       const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
+                                       const int* __restrict__ seq_q_len, int columns) {
+  trigger_dependents();
+  grid_dependency_wait();
+  const int s = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+  const int n = seq_q_len[s];
+  if (n <= 1 || c >= columns) return;
+  float* st = state + (size_t)seq_slot[s] * slot_stride + c;
+  const float* first = qkv + (size_t)seq_q_start[s] * stride + c;
+  float v[HALO > 0 ? HALO : 1];
+#pragma unroll
+  for (int r = 0; r < HALO; r++) {
+    const int idx = n - HALO + r;
+    v[r] = idx >= 0 ? first[(size_t)idx * stride] : st[(size_t)(r + n) * columns];
+  }
+#pragma unroll
+  for (int r = 0; r < HALO; r++) st[(size_t)r * columns] = v[r];
+}
+
+template <typename T>
+int conv_prep_launch(const float* qkv, int stride, const float* taps, float* state, long long slot_stride, int norm,
+                     float eps, void* q_out, void* cache, const int* positions, const int* token_seq, const int* seq_slot,
+                     const int* seq_q_start, const int* seq_q_len, const int* page_indptr, const int* page_ids,
+                     int n_tokens, int n_seqs, int portions, int nh, int nkv, int page_size, int num_pages,
+                     int write_cache, int write_state, int* status, const float* norm_w, const double* freq, int rot_dims,
+                     int rot_pairs, int own_kv, cudaStream_t st) {
+  if (n_tokens <= 0) return 0;
+  if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || page_size <= 0 || norm < 0 || norm > 1) return -2;
+  if (freq != nullptr && (rot_dims < 0 || rot_dims > QK || (rot_dims & 1))) return -2;
+  const int columns = (nh + (own_kv ? nkv : 0)) * MAPS * QK + (own_kv ? nkv * VD : 0);
+  if (HALO > 0 && (state == nullptr || slot_stride < (long long)HALO * columns)) return -2;
+  // few tokens: a block each and their vectors shared out; many: as many as a block takes
+  const int tb = n_tokens < 128 ? 1 : TB;
+  const int gx = (n_tokens + tb - 1) / tb;
+  const int n_vec = (nh + (own_kv ? nkv : 0)) * MAPS + (own_kv ? nkv : 0);
+  int gy = (2 * sm_count() + gx - 1) / gx;
+  const int most = (n_vec + CONV_WARPS - 1) / CONV_WARPS;
+  if (gy > most) gy = most;
+  int rc = launch_pdl(sink_attn_conv_prep_kernel<T>, dim3(gx, gy), dim3(CONV_WARPS * 32), 0, st, qkv, stride, taps, state,
+                      slot_stride, norm, eps, (T*)q_out, (T*)cache, positions, token_seq, seq_slot, seq_q_start,
+                      seq_q_len, page_indptr, page_ids, n_tokens, nh, nkv, page_size, num_pages, write_cache, write_state,
+                      status, norm_w, freq, rot_dims, rot_pairs, own_kv, tb);
+  if (rc != 0 || HALO == 0 || !portions || !write_state || n_seqs <= 0) return rc;
+  if ((columns + 255) / 256 > 65535) return -3;
+  return launch_pdl(sink_conv_state_kernel, dim3(n_seqs, (columns + 255) / 256), dim3(256), 0, st, qkv, stride, state,
+                    slot_stride, seq_slot, seq_q_start, seq_q_len, columns);
+}
+#endif  // TKB_TAPS > 0
+
 // With several maps a head the maps' outputs stay float32 (they are combined before anything rounds them).
 template <typename T> struct OutOf { using type = typename std::conditional<(MAPS > 1), float, T>::type; };
 
@@ -206,7 +457,8 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
                       const int* __restrict__ rows, const float* __restrict__ sinks, int nh, int nkv, int page_size,
                       float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
                       int* __restrict__ status, const float* __restrict__ head_scale, const float* __restrict__ head_bias,
-                      const float* __restrict__ head_slope, int out_stride, float out_scale) {
+                      const float* __restrict__ head_slope, int out_stride, float out_scale,
+                      const float* __restrict__ gate, int gate_stride) {
   using TO = typename OutOf<T>::type;
   __shared__ float qs[WARPS][QK];
   trigger_dependents();
@@ -285,7 +537,7 @@ attn_sink_simt_kernel(const T* __restrict__ q, typename OutOf<T>::type* __restri
         }
       }
     }
-    const float inv_l = (SIGMOID ? 1.f : (l > 0.f ? 1.f / l : 0.f)) * out_scale;
+    const float inv_l = (SIGMOID ? 1.f : (l > 0.f ? 1.f / l : 0.f)) * out_scale * head_gate(gate, gate_stride, t, h);
     TO* orow = out + (size_t)blockIdx.x * out_stride + (size_t)h * VD;
 #pragma unroll
     for (int i = 0; i < DPL; i++) {
@@ -330,17 +582,18 @@ diff_combine_kernel(const float* __restrict__ a, const float* __restrict__ lambd
 }
 
 template <typename T>
-int prep_launch(const float* qkv, int stride, const float* bias, int unit_norm, float eps, void* q_out, void* cache,
+int prep_launch(const float* qkv, int stride, const float* bias, int norm, float eps, void* q_out, void* cache,
                 const int* positions, const int* token_seq, const int* page_indptr, const int* page_ids, int n_tokens,
                 int nh, int nkv, int page_size, int num_pages, int write_cache, int* status, const float* norm_w,
-                const double* freq, int rot_dims, int rot_pairs, int values_are_keys, cudaStream_t st) {
+                const double* freq, int rot_dims, int rot_pairs, int values_are_keys, int own_kv, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || page_size <= 0) return -2;
   if (freq != nullptr && (rot_dims < 0 || rot_dims > QK || (rot_dims & 1))) return -2;
   if (values_are_keys && (QK != VD || MAPS != 1)) return -2;
-  return launch_pdl(sink_attn_prep_kernel<T>, dim3(n_tokens), dim3(256), 0, st, qkv, stride, bias, unit_norm, eps,
+  if (norm < 0 || norm > 2) return -2;
+  return launch_pdl(sink_attn_prep_kernel<T>, dim3(n_tokens), dim3(256), 0, st, qkv, stride, bias, norm, eps,
                     (T*)q_out, (T*)cache, positions, token_seq, page_indptr, page_ids, nh, nkv, page_size, num_pages,
-                    write_cache, status, norm_w, freq, rot_dims, rot_pairs, values_are_keys);
+                    write_cache, status, norm_w, freq, rot_dims, rot_pairs, values_are_keys, own_kv);
 }
 
 template <typename T>
@@ -348,29 +601,29 @@ int attn_launch(const void* q, void* out, const void* cache, const int* token_se
                 const int* page_indptr, const int* page_ids, const int* rows, int n_rows, const float* sinks, int nh,
                 int nkv, int page_size, float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
                 int* status, const float* head_scale, const float* head_bias, const float* head_slope, int out_stride,
-                float out_scale, cudaStream_t st) {
+                float out_scale, const float* gate, int gate_stride, cudaStream_t st) {
   if (n_rows <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || keep_first < 0 || (head_slope != nullptr && !DIST)) return -2;
-  if (out_stride < nh * MAPS * VD) return -2;
+  if (out_stride < nh * MAPS * VD || (gate != nullptr && MAPS != 1)) return -2;
   if (nkv > 65535) return -3;
   return launch_pdl(attn_sink_simt_kernel<T>, dim3(n_rows, nkv), dim3(WARPS * 32), 0, st, (const T*)q,
                     (typename OutOf<T>::type*)out, (const T*)cache, token_seq, positions, page_indptr, page_ids, rows,
                     sinks, nh, nkv, page_size, scale, softcap, window, keep_first, chunk, num_pages, status, head_scale,
-                    head_bias, head_slope, out_stride, out_scale);
+                    head_bias, head_slope, out_stride, out_scale, gate, gate_stride);
 }
 
 }  // namespace
 
 #define TKB_SINK_EXPORTS(SUF, T)                                                                                      \
-  TKB_EXPORT int tkb_sink_attn_prep_##SUF(const float* qkv, int stride, const float* bias, int unit_norm, float eps,  \
+  TKB_EXPORT int tkb_sink_attn_prep_##SUF(const float* qkv, int stride, const float* bias, int norm, float eps,       \
                                           void* q_out, void* cache, const int* positions, const int* token_seq,       \
                                           const int* page_indptr, const int* page_ids, int n_tokens, int nh, int nkv, \
                                           int page_size, int num_pages, int write_cache, int* status,                 \
                                           const float* norm_w, const double* freq, int rot_dims, int rot_pairs,       \
-                                          int values_are_keys, void* st) {                                            \
-    return prep_launch<T>(qkv, stride, bias, unit_norm, eps, q_out, cache, positions, token_seq, page_indptr,         \
+                                          int values_are_keys, int own_kv, void* st) {                                \
+    return prep_launch<T>(qkv, stride, bias, norm, eps, q_out, cache, positions, token_seq, page_indptr,         \
                           page_ids, n_tokens, nh, nkv, page_size, num_pages, write_cache, status, norm_w, freq,       \
-                          rot_dims, rot_pairs, values_are_keys, (cudaStream_t)st);                                    \
+                          rot_dims, rot_pairs, values_are_keys, own_kv, (cudaStream_t)st);                            \
   }                                                                                                                   \
   TKB_EXPORT int tkb_attn_sink_simt_##SUF(const void* q, void* out, const void* cache, const int* token_seq,          \
                                           const int* positions, const int* page_indptr, const int* page_ids,          \
@@ -378,10 +631,10 @@ int attn_launch(const void* q, void* out, const void* cache, const int* token_se
                                           int page_size, float scale, float softcap, int window, int keep_first,      \
                                           int chunk, int num_pages, int* status, const float* head_scale,             \
                                           const float* head_bias, const float* head_slope, int out_stride,            \
-                                          float out_scale, void* st) {                                                \
+                                          float out_scale, const float* gate, int gate_stride, void* st) {            \
     return attn_launch<T>(q, out, cache, token_seq, positions, page_indptr, page_ids, rows, n_rows, sinks, nh, nkv,   \
                           page_size, scale, softcap, window, keep_first, chunk, num_pages, status, head_scale,        \
-                          head_bias, head_slope, out_stride, out_scale, (cudaStream_t)st);                                                                          \
+                          head_bias, head_slope, out_stride, out_scale, gate, gate_stride, (cudaStream_t)st);         \
   }                                                                                                                   \
   TKB_EXPORT int tkb_diff_combine_##SUF(const float* a, const float* lambda, float eps, float mult,                   \
                                         const float* gate, int gate_stride, int gate_off, const int* rows, void* out, \
@@ -394,6 +647,23 @@ int attn_launch(const void* q, void* out, const void* cache, const int* token_se
 
 TKB_SINK_EXPORTS(f32, float)
 TKB_SINK_EXPORTS(bf16, __nv_bfloat16)
+
+#if TKB_TAPS > 0
+#define TKB_SINK_CONV_EXPORT(SUF, T)                                                                                  \
+  TKB_EXPORT int tkb_sink_attn_conv_prep_##SUF(                                                                       \
+      const float* qkv, int stride, const float* taps, float* state, long long slot_stride, int norm, float eps,      \
+      void* q_out, void* cache, const int* positions, const int* token_seq, const int* seq_slot,                      \
+      const int* seq_q_start, const int* seq_q_len, const int* page_indptr, const int* page_ids, int n_tokens,        \
+      int n_seqs, int portions, int nh, int nkv, int page_size, int num_pages, int write_cache, int write_state,      \
+      int* status, const float* norm_w, const double* freq, int rot_dims, int rot_pairs, int own_kv, void* st) {      \
+    return conv_prep_launch<T>(qkv, stride, taps, state, slot_stride, norm, eps, q_out, cache, positions, token_seq,  \
+                               seq_slot, seq_q_start, seq_q_len, page_indptr, page_ids, n_tokens, n_seqs, portions,   \
+                               nh, nkv, page_size, num_pages, write_cache, write_state, status, norm_w, freq,         \
+                               rot_dims, rot_pairs, own_kv, (cudaStream_t)st);                                        \
+  }
+TKB_SINK_CONV_EXPORT(f32, float)
+TKB_SINK_CONV_EXPORT(bf16, __nv_bfloat16)
+#endif
 
 // ------------------------------------------------------------------------------------------------ tensor cores
 #if (TKB_QK % 16 == 0) && (TKB_VD % 16 == 0) && (TKB_QK <= 256) && (TKB_VD <= 256) && (TKB_MAPS != 3)
@@ -605,7 +875,8 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
                        const int* __restrict__ page_ids, int n_seqs, const float* __restrict__ sinks, int nh, int nkv,
                        int ps, float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
                        int* __restrict__ status, const float* __restrict__ head_scale, const float* __restrict__ head_bias,
-                       const float* __restrict__ head_slope, int out_stride, float out_scale) {
+                       const float* __restrict__ head_slope, int out_stride, float out_scale,
+                       const float* __restrict__ gate, int gate_stride) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* bufs = reinterpret_cast<bf16*>(smem_raw);
   trigger_dependents();
@@ -712,7 +983,7 @@ attn_sink_tiles_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restrict
     l[hh] += __shfl_xor_sync(0xffffffffu, l[hh], 2);
     const int r = warp * 16 + g + hh * 8;
     if (r < rows) {
-      const float inv = l[hh] > 0.f ? out_scale / l[hh] : 0.f;
+      const float inv = l[hh] > 0.f ? out_scale / l[hh] * head_gate(gate, gate_stride, start + r0 + r, h) : 0.f;
       auto* orow = out + (size_t)(start + r0 + r) * out_stride + (size_t)h * VD + 2 * t;
 #pragma unroll
       for (int vt = 0; vt < VT; vt++) {
@@ -738,7 +1009,7 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
                         int ps, float scale, float softcap, int window, int keep_first, int chunk, int num_pages,
                         int* __restrict__ status, float* __restrict__ part, const float* __restrict__ head_scale,
                         const float* __restrict__ head_bias, const float* __restrict__ head_slope, int out_stride,
-                        float out_scale) {
+                        float out_scale, const float* __restrict__ gate, int gate_stride) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* bufs = reinterpret_cast<bf16*>(smem_raw);
   trigger_dependents();
@@ -855,7 +1126,8 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
     }
     const int head = (kvh * group + g0 + r) * MAPS + mp;
     if (splits == 1) {
-      out[(size_t)tok * out_stride + (size_t)head * VD + d] = from_float<OutOf<bf16>::type>(ll > 0.f ? acc / ll * out_scale : 0.f);
+      out[(size_t)tok * out_stride + (size_t)head * VD + d] = from_float<OutOf<bf16>::type>(
+          ll > 0.f ? acc / ll * out_scale * head_gate(gate, gate_stride, tok, head) : 0.f);
     } else {  // this split's share: sums relative to its own maximum, for attn_sink_merge
       float* pr = part + (((size_t)s * nhm + head) * splits + split) * (VD + 2);
       pr[d] = acc;
@@ -870,7 +1142,8 @@ attn_sink_single_kernel(const bf16* __restrict__ q, OutOf<bf16>::type* __restric
 // The splits of every single-token request put together: grid (request row, query head).
 __global__ void attn_sink_merge_kernel(const float* __restrict__ part, OutOf<bf16>::type* __restrict__ out,
                                        const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len, int nh,
-                                       int splits, int out_stride, float out_scale) {
+                                       int splits, int out_stride, float out_scale, const float* __restrict__ gate,
+                                       int gate_stride) {
   trigger_dependents();
   grid_dependency_wait();
   const int s = blockIdx.x, head = blockIdx.y;
@@ -880,7 +1153,7 @@ __global__ void attn_sink_merge_kernel(const float* __restrict__ part, OutOf<bf1
   for (int z = 0; z < splits; z++) mm = fmaxf(mm, pr[z * (VD + 2) + VD]);
   float ll = 0.f;
   for (int z = 0; z < splits; z++) ll += exp2f(pr[z * (VD + 2) + VD] - mm) * pr[z * (VD + 2) + VD + 1];
-  const float inv = ll > 0.f ? out_scale / ll : 0.f;
+  const float inv = ll > 0.f ? out_scale / ll * head_gate(gate, gate_stride, seq_q_start[s], head) : 0.f;
   for (int d = threadIdx.x; d < VD; d += blockDim.x) {
     float acc = 0.f;
     for (int z = 0; z < splits; z++) acc += exp2f(pr[z * (VD + 2) + VD] - mm) * pr[z * (VD + 2) + d];
@@ -900,12 +1173,13 @@ TKB_EXPORT int tkb_attn_sink_tc_bf16(const void* q, void* out, const void* cache
                                      const float* sinks, int nh, int nkv, int page_size, float scale, float softcap,
                                      int window, int keep_first, int chunk, int num_pages, int* status, float* part,
                                      int splits, const float* head_scale, const float* head_bias,
-                                     const float* head_slope, int out_stride, float out_scale, void* st) {
+                                     const float* head_slope, int out_stride, float out_scale, const float* gate,
+                                     int gate_stride, void* st) {
   using TO = OutOf<bf16>::type;
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || keep_first < 0 || (head_slope != nullptr && !DIST)) return -2;
   // (the portions' kernel stores pairs of values)
-  if (out_stride < nh * MAPS * VD || (out_stride & 1) || (((uintptr_t)out) & 7)) return -2;
+  if (out_stride < nh * MAPS * VD || (out_stride & 1) || (((uintptr_t)out) & 7) || (gate != nullptr && MAPS != 1)) return -2;
   const int head_tiles = (nh / nkv + 15) / 16;
   if (nh * MAPS > 65535 || nkv * head_tiles > 65535) return -3;
   if (TC_SMEM > 48 * 1024) {
@@ -921,11 +1195,12 @@ TKB_EXPORT int tkb_attn_sink_tc_bf16(const void* q, void* out, const void* cache
     rc = launch_pdl(attn_sink_single_kernel, dim3(n_seqs, nkv * head_tiles, splits), dim3(128), TC_SMEM,
                     (cudaStream_t)st, (const bf16*)q, (TO*)out, (const bf16*)cache, seq_q_start, seq_q_len, seq_kv_len,
                     page_indptr, page_ids, sinks, nh, nkv, head_tiles, page_size, scale, softcap, window, keep_first,
-                    chunk, num_pages, status, part, head_scale, head_bias, head_slope, out_stride, out_scale);
+                    chunk, num_pages, status, part, head_scale, head_bias, head_slope, out_stride, out_scale, gate,
+                    gate_stride);
     if (rc == 0 && splits > 1)
       rc = launch_pdl(attn_sink_merge_kernel, dim3(n_seqs, nh * MAPS), dim3(VD >= 128 ? 128 : 64), 0, (cudaStream_t)st,
                       (const float*)part, (TO*)out, seq_q_start, seq_q_len, nh * MAPS, splits,
-                      out_stride, out_scale);
+                      out_stride, out_scale, gate, gate_stride);
   }
   if (rc != 0 || !portions) return rc;
   const int tiles = n_tokens / KT + n_seqs;  // no step of this shape has more 64-query tiles
@@ -933,7 +1208,7 @@ TKB_EXPORT int tkb_attn_sink_tc_bf16(const void* q, void* out, const void* cache
   return launch_pdl(attn_sink_tiles_kernel, dim3(nh * MAPS, tiles), dim3(128), TC_SMEM, (cudaStream_t)st, (const bf16*)q,
                     (TO*)out, (const bf16*)cache, seq_q_start, seq_q_len, seq_kv_len, page_indptr, page_ids, n_seqs,
                     sinks, nh, nkv, page_size, scale, softcap, window, keep_first, chunk, num_pages, status, head_scale,
-                    head_bias, head_slope, out_stride, out_scale);
+                    head_bias, head_slope, out_stride, out_scale, gate, gate_stride);
 }
 #endif  // tensor-core sizes
 TKB_EXPORT int tkb_attn_sink_has_tc() {

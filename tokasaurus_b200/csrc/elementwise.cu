@@ -827,12 +827,18 @@ TKB_EXPORT int tkb_gelu_tanh_mul_bf16(const void* gu, void* out, int rows, int I
 }
 
 // ------------------------------------------------------------------------------------------------
-// out = gelu(z), the exact (erf) form, for an up product without a gate.  z: float32 slices of a K-split product
+// out = act(z) for an up product without a gate: the exact (erf) GELU, or the square of relu.  z: float32 slices of a K-split product
 // ([n_slices][total], added in slice order), or values in the activation type (z_act).  Four elements a thread where
 // the count allows.
 __device__ __forceinline__ float gelu_erf_f(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
-template <typename T>
-__global__ void gelu_rows_kernel(const float* __restrict__ z, int n_slices, long long stride, const T* __restrict__ z_act,
+constexpr int ROWS_GELU = 0, ROWS_RELU2 = 1;
+template <int ACT> __device__ __forceinline__ float rows_act(float v) {
+  if (ACT == ROWS_GELU) return gelu_erf_f(v);
+  const float r = fmaxf(v, 0.f);
+  return r * r;
+}
+template <typename T, int ACT>
+__global__ void act_rows_kernel(const float* __restrict__ z, int n_slices, long long stride, const T* __restrict__ z_act,
                                  T* __restrict__ out, long long total) {
   trigger_dependents();
   grid_dependency_wait();
@@ -849,7 +855,7 @@ __global__ void gelu_rows_kernel(const float* __restrict__ z, int n_slices, long
           v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
         }
       }
-      store4(out + i, make_float4(gelu_erf_f(v.x), gelu_erf_f(v.y), gelu_erf_f(v.z), gelu_erf_f(v.w)));
+      store4(out + i, make_float4(rows_act<ACT>(v.x), rows_act<ACT>(v.y), rows_act<ACT>(v.z), rows_act<ACT>(v.w)));
     }
     return;
   }
@@ -861,27 +867,52 @@ __global__ void gelu_rows_kernel(const float* __restrict__ z, int n_slices, long
       v = z[i];
       for (int s = 1; s < n_slices; s++) v += z[(size_t)s * stride + i];
     }
-    out[i] = from_float<T>(gelu_erf_f(v));
+    out[i] = from_float<T>(rows_act<ACT>(v));
   }
 }
-template <typename T>
-static int gelu_rows_launch(const float* z, int n_slices, long long stride, const void* z_act, void* out, long long total,
-                            cudaStream_t st) {
+template <typename T, int ACT>
+static int act_rows_launch(const float* z, int n_slices, long long stride, const void* z_act, void* out, long long total,
+                           cudaStream_t st) {
   if (total <= 0) return 0;
   if ((z == nullptr) == (z_act == nullptr) || (z != nullptr && n_slices < 1)) return -2;
   long long blocks = (total / 4 + 255) / 256;
   if (blocks > sm_count() * 16) blocks = sm_count() * 16;
   if (blocks < 1) blocks = 1;
-  return launch_pdl(gelu_rows_kernel<T>, dim3((int)blocks), dim3(256), 0, st, z, n_slices, stride, (const T*)z_act, (T*)out,
-                    total);
+  return launch_pdl(act_rows_kernel<T, ACT>, dim3((int)blocks), dim3(256), 0, st, z, n_slices, stride, (const T*)z_act,
+                    (T*)out, total);
 }
-TKB_EXPORT int tkb_gelu_rows_f32(const float* z, int n_slices, long long stride, const void* z_act, void* out,
-                                 long long total, void* st) {
-  return gelu_rows_launch<float>(z, n_slices, stride, z_act, out, total, (cudaStream_t)st);
+#define TKB_ACT_ROWS_EXPORT(NAME, T, ACT)                                                                       \
+  TKB_EXPORT int NAME(const float* z, int n_slices, long long stride, const void* z_act, void* out,             \
+                      long long total, void* st) {                                                              \
+    return act_rows_launch<T, ACT>(z, n_slices, stride, z_act, out, total, (cudaStream_t)st);                   \
+  }
+TKB_ACT_ROWS_EXPORT(tkb_gelu_rows_f32, float, ROWS_GELU)
+TKB_ACT_ROWS_EXPORT(tkb_gelu_rows_bf16, __nv_bfloat16, ROWS_GELU)
+TKB_ACT_ROWS_EXPORT(tkb_relu2_rows_f32, float, ROWS_RELU2)
+TKB_ACT_ROWS_EXPORT(tkb_relu2_rows_bf16, __nv_bfloat16, ROWS_RELU2)
+
+// x = cap * tanh(x / cap) in place on float32 values (an output head's logits).
+__global__ void soft_cap_kernel(float* __restrict__ x, float cap, long long total) {
+  trigger_dependents();
+  grid_dependency_wait();
+  const float inv = 1.f / cap;
+  const long long step = (long long)gridDim.x * blockDim.x * 4;
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < total; i += step) {
+    if (i + 4 <= total && ((uintptr_t)x & 15) == 0) {
+      const float4 v = load4(x + i);
+      store4(x + i, make_float4(cap * tanhf(v.x * inv), cap * tanhf(v.y * inv), cap * tanhf(v.z * inv), cap * tanhf(v.w * inv)));
+    } else {
+      for (long long j = i; j < total && j < i + 4; j++) x[j] = cap * tanhf(x[j] * inv);
+    }
+  }
 }
-TKB_EXPORT int tkb_gelu_rows_bf16(const float* z, int n_slices, long long stride, const void* z_act, void* out,
-                                  long long total, void* st) {
-  return gelu_rows_launch<__nv_bfloat16>(z, n_slices, stride, z_act, out, total, (cudaStream_t)st);
+TKB_EXPORT int tkb_soft_cap(float* x, float cap, long long total, void* st) {
+  if (total <= 0) return 0;
+  if (!(cap > 0.f)) return -2;
+  long long blocks = (total / 4 + 255) / 256;
+  if (blocks > sm_count() * 8) blocks = sm_count() * 8;
+  if (blocks < 1) blocks = 1;
+  return launch_pdl(soft_cap_kernel, dim3((int)blocks), dim3(256), 0, (cudaStream_t)st, x, cap, total);
 }
 
 // ------------------------------------------------------------------------------------------------

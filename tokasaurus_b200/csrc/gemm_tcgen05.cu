@@ -12,7 +12,7 @@
 //            tile fill the second accumulator buffer.
 // Epilogues: bfloat16 store; or, for a weight that interleaves gate and up rows in groups of 8,
 // silu(gate) * up as bfloat16 [M, N/2] (the activation pass over memory disappears); or, for an ungated weight, the
-// exact (erf) GELU of the product.
+// exact (erf) GELU of the product, or the square of its relu.
 //
 // No load uses cluster multicast.  Every wait on an mbarrier is bounded: after the limit the block sets
 // TKB_STATUS_WAIT_TIMEOUT in the status word, stops waiting, frees its tensor memory and returns.
@@ -157,6 +157,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 const float v = __uint_as_float(r[jj]);
                 r[jj] = __float_as_uint(0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
               }
+            } else if (plain_act == 2) {  // the square of relu
+#pragma unroll
+              for (int jj = 0; jj < 32; jj++) {
+                const float v = fmaxf(__uint_as_float(r[jj]), 0.f);
+                r[jj] = __float_as_uint(v * v);
+              }
             }
             const int n = n0 + c0;
             bf16* dst = out + (size_t)row * ldo + n;
@@ -250,12 +256,13 @@ int launch(const void* A, int lda, const void* W, int ldw, void* out, int ldo, i
 }  // namespace
 
 // out[M, N] (bfloat16, row stride ldo) = A[M, K] . W[N, K]^T.  gated == 1: W interleaves gate/up rows in groups of
-// 8 and out is [M, N/2] = silu(gate) * up; gated == 2: ungated, the exact GELU of every result.  K and the row strides must be multiples of 8 elements and the base
+// 8 and out is [M, N/2] = silu(gate) * up; gated == 2: ungated, the exact GELU of every result; gated == 3: ungated, relu(result)^2.  K and the row strides must be multiples of 8 elements and the base
 // addresses 16-byte aligned (what a TMA descriptor asks for); N a multiple of 16 for the gated form.
 TKB_EXPORT int tkb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M, int N,
                                      int K, int gated, int* status, void* st_) {
-  const int plain_act = gated == 2 ? 1 : 0;
-  if (gated == 2) gated = 0;
+  const int plain_act = gated >= 2 ? gated - 1 : 0;
+  if (gated < 0 || gated > 3) return -2;
+  if (gated >= 2) gated = 0;
   cudaStream_t st = (cudaStream_t)st_;
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (lda & 7) || (ldw & 7) || (((uintptr_t)A) & 15) || (((uintptr_t)W) & 15)) return -2;
@@ -287,13 +294,15 @@ TKB_EXPORT int tkb_gemm_tcgen05_clamped_bf16(const void* A, int lda, const void*
 // Grouped form: W is [groups * N, K], rows g * N .. (g + 1) * N the weights of group g, and row tile i of A (128
 // rows) multiplies the weights of group tile_group[i] (a device array of ceil(M / 128) entries; -1: the tile is
 // nobody's and is left out).  The caller orders A's rows by group and starts every group on a tile boundary.
-// gated: 0 plain, 1 silu(gate) * up over interleaved rows, 2 plain with the exact GELU of every result.
+// gated: 0 plain, 1 silu(gate) * up over interleaved rows, 2 plain with the exact GELU of every result,
+// 3 plain with relu(result)^2.
 // row_scale (gated == 1; float32 [M] or null): row i of A counts row_scale[i] times, applied to the accumulator.
 TKB_EXPORT int tkb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M,
                                              int N, int K, int gated, const int* tile_group, int groups,
                                              const float* row_scale, int* status, void* st_) {
-  const int plain_act = gated == 2 ? 1 : 0;
-  if (gated == 2) gated = 0;
+  const int plain_act = gated >= 2 ? gated - 1 : 0;
+  if (gated < 0 || gated > 3) return -2;
+  if (gated >= 2) gated = 0;
   cudaStream_t st = (cudaStream_t)st_;
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (lda & 7) || (ldw & 7) || (((uintptr_t)A) & 15) || (((uintptr_t)W) & 15)) return -2;

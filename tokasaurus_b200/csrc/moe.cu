@@ -8,6 +8,8 @@
 // neighbours only (a group scores the sum of its two largest choice scores); the weights are the chosen experts' s over
 // their sum (+ 1e-20), times a scale, or (renorm == 0) s times a scale as it is.  A second kind of expert:
 // down(gelu(up h)) with the exact (erf) GELU, no gate.
+// A third: down(relu(up h)^2), no gate.  A third way of choosing (moe_table): no router, a table gives every token id its
+// experts, each of weight 1 / top.
 // Weights on the way IN: with pair_scale (float32, one number a (token, choice) pair) an expert reads w * h instead of h,
 // and the outputs are added up unweighed.  A factor on a row of the operand is a factor on the row of the product, so
 // the first product's sums are multiplied before the activation sees them.
@@ -232,6 +234,32 @@ moe_choose_scored_kernel(const float* __restrict__ z_all, const float* __restric
   for (int k = lane; k < top; k += 32) top_w[(size_t)t * top + k] *= f;
 }
 
+// No router: token t's experts are row id(t) of an int32 table [V, top], each of weight 1 / top.  The id is found as the
+// embedding finds it (ids[t] < 0: the token the request sampled last).  rows names the tokens of a cut-down set of rows
+// (null: row r is token r).  Padding tokens, and ids outside the table (they set the status flag), choose nothing.
+__global__ void moe_table_kernel(const int* __restrict__ table, int V, int E, int top, const int* __restrict__ ids,
+                                 const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
+                                 const int* __restrict__ last_token, const int* __restrict__ rows,
+                                 int* __restrict__ top_idx, float* __restrict__ top_w, int n_rows, int* __restrict__ status) {
+  trigger_dependents();
+  grid_dependency_wait();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n_rows * top) return;
+  const int r = i / top, k = i - r * top;
+  const int t = rows != nullptr ? rows[r] : r;
+  const int s = token_seq[t];
+  int e = -1;
+  if (s >= 0) {
+    int id = ids[t];
+    if (id < 0) id = last_token[seq_slot[s]];
+    if (id >= 0 && id < V) e = table[(size_t)id * top + k];
+    else atomicOr(status, TKB_STATUS_BAD_TOKEN_ID);
+  }
+  const bool live = e >= 0 && e < E;
+  top_idx[i] = live ? e : -1;
+  top_w[i] = live ? 1.f / (float)top : 0.f;
+}
+
 // One block: offsets[e] .. is expert e's span of the ordering; order[p] is the (token, choice) pair at place p
 // (token * top + choice), place_of[pair] its place (-1 for a padding token's pairs).  pad > 1: every span starts at
 // a multiple of pad (the tensor-core product's row tile), offsets[e + 1] - offsets[e] is then the span with its
@@ -313,10 +341,11 @@ __global__ void moe_gather_kernel(const T* __restrict__ src, const int* __restri
 //   plain:  C[p, n] = A[src(p), :] . W[e][n, :]                      (C float32 [places, N])
 //   gated:  C[p, n] = silu(A[src(p), :] . W[e][n, :]) * (A[src(p), :] . W[e][N + n, :])      (W[e] is [2N, K])
 //   gelu:   C[p, n] = gelu(A[src(p), :] . W[e][n, :]), the exact (erf) form, in A's type
+//   relu2:  C[p, n] = relu(A[src(p), :] . W[e][n, :])^2 in A's type
 // src(p) = order[p] / top if `order` is given (rows of the step's tokens), else p.  Block (x, y): column tile x of the
 // y-th row tile, counted over the experts' spans in turn; blocks beyond the last tile leave at once.
 constexpr int BM = 64, BN = 64, BK = 16;
-constexpr int ACT_NONE = 0, ACT_GATED = 1, ACT_GELU = 2, ACT_CLAMPED = 3;
+constexpr int ACT_NONE = 0, ACT_GATED = 1, ACT_GELU = 2, ACT_CLAMPED = 3, ACT_RELU2 = 4;
 // the clamped gated unit: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha g) * (u + 1)
 __device__ __forceinline__ float clamped_unit(float gate, float up, float limit, float alpha) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
@@ -414,6 +443,7 @@ moe_gemm_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC*
       if (ACT == ACT_CLAMPED) v = clamped_unit(v, acu[i][j], limit, alpha);
       else if (GATED) v = v / (1.f + expf(-v)) * acu[i][j];
       if (ACT == ACT_GELU) v = gelu_erf_f(v);
+      if (ACT == ACT_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
       C[(size_t)p * ldc + n] = from_float<TC>(v);
     }
   }
@@ -521,6 +551,7 @@ moe_gemv_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ W, TC*
               v = ACT == ACT_CLAMPED ? clamped_unit(v, u, limit, alpha) : v / (1.f + expf(-v)) * u;
             }
             if (ACT == ACT_GELU) v = gelu_erf_f(v);
+            if (ACT == ACT_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
             const int f = f0 + j;
             if (lane == 0 && f < N) C[(size_t)(r0 + r) * ldc + f] = from_float<TC>(v);
           }
@@ -620,6 +651,15 @@ int combine_launch(const void* y, const int* place_of, const float* top_w, const
 
 }  // namespace
 
+TKB_EXPORT int tkb_moe_table(const int* table, int V, int E, int top, const int* ids, const int* token_seq,
+                             const int* seq_slot, const int* last_token, const int* rows, int* top_idx, float* top_w,
+                             int n_rows, int* status, void* st) {
+  if (n_rows <= 0) return 0;
+  if (V <= 0 || E <= 0 || top <= 0 || top > E || (long long)n_rows * top > 0x7fffffffll - 256) return -2;
+  return launch_pdl(moe_table_kernel, dim3((n_rows * top + 255) / 256), dim3(256), 0, (cudaStream_t)st, table, V, E, top,
+                    ids, token_seq, seq_slot, last_token, rows, top_idx, top_w, n_rows, status);
+}
+
 TKB_EXPORT int tkb_moe_order(const int* top_idx, int n_pairs, int E, int top, int pad, int* offsets, int* order,
                              int* place_of, int* tile_group, int n_tiles, int* src_token, int cap, void* st) {
   if (n_pairs <= 0) return 0;
@@ -658,6 +698,10 @@ TKB_EXPORT int tkb_moe_order(const int* top_idx, int n_pairs, int E, int top, in
   TKB_EXPORT int tkb_moe_gemm_gelu_##SUF(const void* A, int lda, const void* W, void* C, int ldc, const int* offsets,  \
                                          const int* order, int top, int n_places, int E, int N, int K, void* st) {     \
     return gemm_launch<T, T, ACT_GELU>(A, lda, W, C, ldc, offsets, order, top, n_places, E, N, K, (cudaStream_t)st);   \
+  }                                                                                                                    \
+  TKB_EXPORT int tkb_moe_gemm_relu2_##SUF(const void* A, int lda, const void* W, void* C, int ldc, const int* offsets, \
+                                          const int* order, int top, int n_places, int E, int N, int K, void* st) {    \
+    return gemm_launch<T, T, ACT_RELU2>(A, lda, W, C, ldc, offsets, order, top, n_places, E, N, K, (cudaStream_t)st);  \
   }                                                                                                                    \
   TKB_EXPORT int tkb_moe_route_scored_##SUF(const void* h, const float* wr, const float* br, const float* correction,  \
                                             const int* token_seq, int* top_idx, float* top_w, float* logits,           \

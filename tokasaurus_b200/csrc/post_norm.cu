@@ -4,6 +4,9 @@
 //   scaled_norm_add   x += mult * scale[c] * w[c] * (y + bias)[c] / sqrt(mean((y + bias)^2) + eps)   (x float32, in
 //                     place), and the new x in the activation type for the sublayer that reads it next; y whole
 //                     rows or the float32 slices of a K-split product
+//   norm_add_norm     x += w1 * N(y), then out = w2 * N(x): the norm on a sublayer's output, the residual sum and the norm
+//                     ahead of the next sublayer in one pass (x float32, in place; y float32 rows or slices; each N with
+//                     an eps of its own)
 //   cast_rows         float32 rows in the activation type
 //   add_sinusoid      x[t][2i] += sin(p_t * f_i),  x[t][2i+1] += cos(p_t * f_i)   (f_i a float64 table)
 //   clamped_glu       g = min(gate, L), u = clamp(up, -L, L), out = g * sigmoid(alpha * g) * (u + 1)
@@ -61,6 +64,142 @@ scaled_norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, int n
     x[row + c] = nx;
     if (h_out) h_out[row + c] = from_float<T>(nx);
   }
+}
+
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<uint32_t*>(&a);
+  u.y = *reinterpret_cast<uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+// The pair of norms, four values a thread and step; V4 steps cover a row, whose values stay in registers from the first
+// load to the last store.  (The slices of a K-split product are added in slice order, four loads in flight.)
+template <typename T, int V4>
+__global__ void __launch_bounds__(512)
+norm_add_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, int n_slices, long long slice_stride,
+                         const float* __restrict__ w1, float eps1, const float* __restrict__ w2, float eps2,
+                         T* __restrict__ out, int H) {
+  __shared__ float red[33];
+  trigger_dependents();
+  const size_t row = (size_t)blockIdx.x * H;
+  const int n4 = H >> 2;
+  grid_dependency_wait();
+  float4 v[V4], xv[V4];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < V4; k++) {
+    const int i4 = threadIdx.x + k * blockDim.x;
+    if (i4 < n4) {
+      v[k] = ld4(y + row + 4 * i4);
+      xv[k] = ld4(x + row + 4 * i4);
+    } else {
+      v[k] = xv[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
+  for (int s0 = 1; s0 < n_slices; s0 += 4) {
+#pragma unroll
+    for (int k = 0; k < V4; k++) {
+      const int i4 = threadIdx.x + k * blockDim.x;
+      if (i4 < n4) {
+        float4 q[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+          q[j] = s0 + j < n_slices ? ld4(y + (size_t)(s0 + j) * slice_stride + row + 4 * i4) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+          v[k].x += q[j].x; v[k].y += q[j].y; v[k].z += q[j].z; v[k].w += q[j].w;
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < V4; k++) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+  const float r1 = rsqrtf(block_sum(ss, red) / (float)H + eps1);
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < V4; k++) {
+    const int i4 = threadIdx.x + k * blockDim.x;
+    if (i4 < n4) {
+      const float4 g = ld4(w1 + 4 * i4);
+      float4 u = xv[k];
+      u.x = fmaf(v[k].x * r1, g.x, u.x);
+      u.y = fmaf(v[k].y * r1, g.y, u.y);
+      u.z = fmaf(v[k].z * r1, g.z, u.z);
+      u.w = fmaf(v[k].w * r1, g.w, u.w);
+      st4(x + row + 4 * i4, u);
+      xv[k] = u;
+      ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+    }
+  }
+  const float r2 = rsqrtf(block_sum(ss, red) / (float)H + eps2);
+#pragma unroll
+  for (int k = 0; k < V4; k++) {
+    const int i4 = threadIdx.x + k * blockDim.x;
+    if (i4 < n4) {
+      const float4 g = ld4(w2 + 4 * i4), u = xv[k];
+      st4(out + row + 4 * i4, make_float4(u.x * r2 * g.x, u.y * r2 * g.y, u.z * r2 * g.z, u.w * r2 * g.w));
+    }
+  }
+}
+
+// Any width: a thread reads back what it wrote itself.
+template <typename T>
+__global__ void __launch_bounds__(512)
+norm_add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int n_slices, long long slice_stride,
+                     const float* __restrict__ w1, float eps1, const float* __restrict__ w2, float eps2,
+                     T* __restrict__ out, int H) {
+  __shared__ float red[33];
+  trigger_dependents();
+  grid_dependency_wait();
+  const size_t row = (size_t)blockIdx.x * H;
+  auto value = [&](int c) {
+    float v = y[row + c];
+    for (int s = 1; s < n_slices; s++) v += y[(size_t)s * slice_stride + row + c];
+    return v;
+  };
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < H; c += blockDim.x) {
+    const float v = value(c);
+    ss = fmaf(v, v, ss);
+  }
+  const float r1 = rsqrtf(block_sum(ss, red) / (float)H + eps1);
+  ss = 0.f;
+  for (int c = threadIdx.x; c < H; c += blockDim.x) {
+    const float nx = fmaf(value(c) * r1, w1[c], x[row + c]);
+    x[row + c] = nx;
+    ss = fmaf(nx, nx, ss);
+  }
+  const float r2 = rsqrtf(block_sum(ss, red) / (float)H + eps2);
+  for (int c = threadIdx.x; c < H; c += blockDim.x) out[row + c] = from_float<T>(x[row + c] * r2 * w2[c]);
+}
+
+template <typename T>
+int norm_add_norm_launch(float* x, const float* y, int n_slices, long long slice_stride, const float* w1, float eps1,
+                         const float* w2, float eps2, void* out, int rows, int H, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || n_slices < 1 || y == nullptr) return -2;
+  const bool aligned = ((((uintptr_t)x) | ((uintptr_t)y) | ((uintptr_t)w1) | ((uintptr_t)w2) | ((uintptr_t)out)) & 15) == 0;
+  if ((H & 3) == 0 && (slice_stride & 3) == 0 && aligned && H <= 512 * 4 * 8) {
+    const int n4 = H >> 2;
+    // few rows: many threads a row, they hide the latency; many rows: 256 threads, so that an SM holds several rows
+    int threads = 32;
+    while (threads < n4 && threads < (rows < 592 || n4 > 2048 ? 512 : 256)) threads <<= 1;
+    const int steps = (n4 + threads - 1) / threads;
+#define TKB_NAN(V4)                                                                                                    \
+  return launch_pdl(norm_add_norm_vec_kernel<T, V4>, dim3(rows), dim3(threads), 0, st, x, y, n_slices, slice_stride,   \
+                    w1, eps1, w2, eps2, (T*)out, H)
+    if (steps <= 1) TKB_NAN(1);
+    if (steps <= 2) TKB_NAN(2);
+    if (steps <= 4) TKB_NAN(4);
+    TKB_NAN(8);
+#undef TKB_NAN
+  }
+  return launch_pdl(norm_add_norm_kernel<T>, dim3(rows), dim3(row_threads(H)), 0, st, x, y, n_slices, slice_stride, w1,
+                    eps1, w2, eps2, (T*)out, H);
 }
 
 template <typename T>
@@ -218,6 +357,11 @@ gated_group_norm_kernel(const float* __restrict__ y, int y_stride, const float* 
     if (H <= 0 || n_slices < 1) return -2;                                                                            \
     return launch_pdl(scaled_norm_add_kernel<T>, dim3(rows), dim3(row_threads(H)), 0, (cudaStream_t)st, x, y,         \
                       n_slices, slice_stride, bias, w, scale, mult, eps, (T*)h_out, H);                               \
+  }                                                                                                                   \
+  TKB_EXPORT int tkb_norm_add_norm_##SUF(float* x, const float* y, int n_slices, long long slice_stride,              \
+                                         const float* w1, float eps1, const float* w2, float eps2, void* out,         \
+                                         int rows, int H, void* st) {                                                 \
+    return norm_add_norm_launch<T>(x, y, n_slices, slice_stride, w1, eps1, w2, eps2, out, rows, H, (cudaStream_t)st); \
   }                                                                                                                   \
   TKB_EXPORT int tkb_cast_rows_##SUF(const float* x, void* out, long long n, void* st) {                              \
     if (n <= 0) return 0;                                                                                             \

@@ -328,17 +328,31 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, interleave: int = 0, act:
     _check(f(_ptr(gate_up), _ptr(out), c_int(rows), c_int(two_i // 2), c_int(interleave), _stream()), "silu_mul")
 
 
-def gelu_rows(z: torch.Tensor, out: torch.Tensor) -> None:
-    """out [rows, I] = gelu(z), the exact (erf) form; z [rows, I] in out's dtype or float32, or float32 slices
+# ungated activations (an up product without a gate) and their number as a product's epilogue: "gelu" the exact (erf)
+# GELU, "relu2" the square of relu
+UNGATED_ACTS = {"gelu": 2, "relu2": 3}
+
+
+def act_rows(z: torch.Tensor, out: torch.Tensor, act: str) -> None:
+    """out [rows, I] = act(z) (``UNGATED_ACTS``); z [rows, I] in out's dtype or float32, or float32 slices
     [slices, rows, I] of a split product, added in slice order."""
     _need_cuda(z, out)
-    _need(z.is_contiguous() and out.is_contiguous() and tuple(z.shape[-2:]) == tuple(out.shape), "gelu_rows: shapes")
+    _need(act in UNGATED_ACTS, f"act_rows: the activation is one of {sorted(UNGATED_ACTS)}, not {act!r}")
+    _need(z.is_contiguous() and out.is_contiguous() and tuple(z.shape[-2:]) == tuple(out.shape), "act_rows: shapes")
     f32 = z.dtype == torch.float32
-    _need(f32 or (z.dtype == out.dtype and z.dim() == 2), "gelu_rows: z float32 or in out's type")
+    _need(f32 or (z.dtype == out.dtype and z.dim() == 2), "act_rows: z float32 or in out's type")
     n = z.shape[0] if z.dim() == 3 else 1
-    _check(_fn(_libs.get("elementwise.cu"), f"tkb_gelu_rows_{_suffix(out.dtype)}")(
+    _check(_fn(_libs.get("elementwise.cu"), f"tkb_{act}_rows_{_suffix(out.dtype)}")(
         _ptr(z if f32 else None), c_int(n), ctypes.c_longlong(out.numel()), _ptr(None if f32 else z), _ptr(out),
-        ctypes.c_longlong(out.numel()), _stream()), "gelu_rows")
+        ctypes.c_longlong(out.numel()), _stream()), "act_rows")
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> None:
+    """x = cap * tanh(x / cap) in place, float32."""
+    _need_cuda(x)
+    _need(x.dtype == torch.float32 and x.is_contiguous() and cap > 0, "soft_cap: contiguous float32, a positive cap")
+    _check(_fn(_libs.get("elementwise.cu"), "tkb_soft_cap")(_ptr(x), c_float(cap), ctypes.c_longlong(x.numel()), _stream()),
+           "soft_cap")
 
 
 def gather_rows(src: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
@@ -630,20 +644,21 @@ def can_use_tcgen05(a: torch.Tensor, w: torch.Tensor) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor, gated: bool = False, gelu: bool = False) -> torch.Tensor:
+def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor, gated: bool = False, act: str | None = None) -> torch.Tensor:
     """a[M, K] @ w[N, K]^T in bfloat16 on the tcgen05 tensor cores (TMA-fed, accumulator in tensor memory).
     ``gated``: ``w`` interleaves gate/up rows (``interleave_gate_up``); the result is silu(gate)*up [M, N/2].
-    ``gelu`` (ungated): the exact GELU of every result in the epilogue.
+    ``act`` (ungated): an activation of every result in the epilogue (``UNGATED_ACTS``).
     ``status``: the device status word; a bounded wait that runs out sets its bit 4."""
     _need_cuda(a, w, status)
     _need(can_use_tcgen05(a, w), "gemm_tcgen05: bfloat16 operands, K and strides multiples of 8, 16-byte aligned")
     M, K = a.shape
     N = w.shape[0]
-    _need(w.shape[1] == K and (not gated or N % 16 == 0) and not (gated and gelu), "gemm_tcgen05: shapes")
+    _need(w.shape[1] == K and (not gated or N % 16 == 0) and not (gated and act), "gemm_tcgen05: shapes")
+    _need(act is None or act in UNGATED_ACTS, f"gemm_tcgen05: unknown activation {act!r}")
     out = torch.empty((M, N // 2 if gated else N), dtype=torch.bfloat16, device=a.device)
     _check(_fn(_libs.get("gemm_tcgen05.cu"), "tkb_gemm_tcgen05_bf16")(
         _ptr(a), c_int(a.stride(0)), _ptr(w), c_int(w.stride(0)), _ptr(out), c_int(out.stride(0)), c_int(M), c_int(N),
-        c_int(K), c_int(1 if gated else (2 if gelu else 0)), _ptr(status), _stream()), "gemm_tcgen05")
+        c_int(K), c_int(1 if gated else (UNGATED_ACTS[act] if act else 0)), _ptr(status), _stream()), "gemm_tcgen05")
     return out
 
 
@@ -1009,6 +1024,25 @@ def moe_route(h: torch.Tensor, router_w: torch.Tensor, router_b: torch.Tensor | 
              c_int(H), c_int(E), c_int(top), c_int(1 if over_all else 0), c_float(scale), _stream()), "moe_route")
 
 
+def moe_table(table: torch.Tensor, n_experts: int, ids: torch.Tensor, token_seq: torch.Tensor, seq_slot: torch.Tensor,
+              last_token: torch.Tensor, rows: torch.Tensor | None, top_idx: torch.Tensor, top_w: torch.Tensor,
+              status: torch.Tensor) -> None:
+    """Experts by token id: top_idx[r] = table[id of row r's token], top_w[r] = 1 / top; table int32 [V, top].  ids[t] < 0
+    takes last_token[seq_slot[token_seq[t]]], as in the embedding; ``rows`` int32 names the tokens of the rows (None: row r
+    is token r).  Padding tokens choose nothing."""
+    _need_cuda(table, ids, token_seq, seq_slot, last_token, rows, top_idx, top_w, status)
+    n, top = top_idx.shape
+    _need(table.dtype == torch.int32 and table.is_contiguous() and table.dim() == 2 and table.shape[1] == top, "moe_table: table int32 [V, top]")
+    _need(ids.dtype == torch.int32 and token_seq.dtype == torch.int32, "moe_table: ids, token_seq int32")
+    _need((rows is None and ids.numel() >= n and token_seq.numel() >= n)
+          or (rows is not None and rows.dtype == torch.int32 and rows.numel() == n), "moe_table: a token for every row")
+    _need(top_idx.dtype == torch.int32 and top_w.dtype == torch.float32 and tuple(top_w.shape) == (n, top)
+          and top_idx.is_contiguous() and top_w.is_contiguous(), "moe_table: outputs [rows, top]")
+    _check(_fn(_libs.get("moe.cu"), "tkb_moe_table")(
+        _ptr(table), c_int(table.shape[0]), c_int(n_experts), c_int(top), _ptr(ids), _ptr(token_seq), _ptr(seq_slot),
+        _ptr(last_token), _ptr(rows), _ptr(top_idx), _ptr(top_w), c_int(n), _ptr(status), _stream()), "moe_table")
+
+
 def moe_logits(h: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None) -> None:
     """out [T, E] = h @ w^T (+ bias) with float32 weights w [E, H], float32 sums: the router's first kernel alone, for
     other small products that want float32 (a gate of one number a token)."""
@@ -1063,12 +1097,12 @@ def moe_gather(src: torch.Tensor, src_token: torch.Tensor, out: torch.Tensor, or
 
 
 def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, status: torch.Tensor,
-                         gated: bool = False, gelu: bool = False, clamp: tuple[float, float] | None = None,
+                         gated: bool = False, act: str | None = None, clamp: tuple[float, float] | None = None,
                          row_scale: torch.Tensor | None = None) -> torch.Tensor:
     """Row tile i (128 rows) of a[M, K] times the weights w[tile_group[i]] of w [groups, N, K], bfloat16 on the tcgen05
     tensor cores; tiles with tile_group[i] < 0 are left out (their rows of the result are not written).
     ``gated``: every group's rows interleave gate and up (``interleave_gate_up``); the result is [M, N / 2].
-    ``gelu`` (ungated): the exact GELU of every result in the epilogue.  ``clamp`` = (limit, alpha), with ``gated``:
+    ``act`` (ungated): an activation of every result in the epilogue (``UNGATED_ACTS``).  ``clamp`` = (limit, alpha), with ``gated``:
     the clamped unit g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), in the SiLU's
     place.  ``row_scale`` float32 [M] (``gated``, no ``clamp``): row i of ``a`` counts row_scale[i] times."""
     _need_cuda(a, w, tile_group, status, row_scale)
@@ -1079,7 +1113,7 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Ten
     M = a.shape[0]
     _need(tile_group.dtype == torch.int32 and tile_group.numel() * 128 >= M, "gemm_tcgen05_grouped: a group for every row tile")
     _need(not gated or N % 16 == 0, "gemm_tcgen05_grouped: gated rows come in groups of 16")
-    _need(not (gated and gelu), "gemm_tcgen05_grouped: the GELU epilogue is the ungated form's")
+    _need(act is None or (not gated and act in UNGATED_ACTS), "gemm_tcgen05_grouped: plain activations are the ungated form's")
     out = torch.empty((M, N // 2 if gated else N), dtype=torch.bfloat16, device=a.device)
     if clamp is not None:
         _need(gated and clamp[0] > 0, "gemm_tcgen05_grouped: the clamped unit is a gated form with a positive limit")
@@ -1089,17 +1123,17 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Ten
         return out
     _check(_fn(_libs.get("gemm_tcgen05.cu"), "tkb_gemm_tcgen05_grouped_bf16")(
         _ptr(a), c_int(a.stride(0)), _ptr(w), c_int(K), _ptr(out), c_int(out.stride(0)), c_int(M), c_int(N), c_int(K),
-        c_int(1 if gated else (2 if gelu else 0)), _ptr(tile_group), c_int(G), _ptr(row_scale), _ptr(status), _stream()),
+        c_int(1 if gated else (UNGATED_ACTS[act] if act else 0)), _ptr(tile_group), c_int(G), _ptr(row_scale), _ptr(status), _stream()),
         "gemm_tcgen05_grouped")
     return out
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor | None,
-             top: int, gated: bool, gelu: bool = False, clamp: tuple[float, float] | None = None,
+             top: int, gated: bool, act: str | None = None, clamp: tuple[float, float] | None = None,
              pair_scale: torch.Tensor | None = None) -> None:
     """The experts' products over the ordering.  w [E, N (2N if gated), K]; a [., K]; row p of ``out`` is made from
     row order[p] // top of ``a`` (row p if ``order`` is None) with the weights of the expert whose span holds p.
-    gated: out = silu(a w_gate^T) * (a w_up^T) in a's type [places, N]; gelu: out = gelu(a w^T) (exact) in a's type;
+    gated: out = silu(a w_gate^T) * (a w_up^T) in a's type [places, N]; ``act`` (``UNGATED_ACTS``): out = act(a w^T) in a's type;
     else float32 [places, N].  ``clamp`` = (limit, alpha), with ``gated``: the clamped unit
     g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), in the SiLU's place.
     ``pair_scale`` float32 [pairs] (``gated``, no ``clamp``, with ``order``): the row of pair order[p] counts so many times."""
@@ -1110,14 +1144,14 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch
     E, NN, K = w.shape
     N = NN // 2 if gated else NN
     _need(a.dtype == w.dtype and a.stride(1) == 1 and a.shape[1] == K and w.is_contiguous(), "moe_gemm: operands")
-    _need(not (gated and gelu), "moe_gemm: gated or gelu")
-    _need(out.shape[1] == N and out.stride(1) == 1 and out.dtype == (a.dtype if (gated or gelu) else torch.float32), "moe_gemm: out")
+    _need(act is None or (not gated and act in UNGATED_ACTS), "moe_gemm: gated, or a plain activation")
+    _need(out.shape[1] == N and out.stride(1) == 1 and out.dtype == (a.dtype if (gated or act) else torch.float32), "moe_gemm: out")
     if clamp is not None:
         _check(_fn(_libs.get("moe.cu"), f"tkb_moe_gemm_clamped_{_suffix(a.dtype)}")(
             _ptr(a), c_int(a.stride(0)), _ptr(w), _ptr(out), c_int(out.stride(0)), _ptr(offsets), _ptr(order), c_int(top),
             c_int(out.shape[0]), c_int(E), c_int(N), c_int(K), c_float(clamp[0]), c_float(clamp[1]), _stream()), "moe_gemm")
         return
-    name = f"tkb_moe_gemm_{'gated_' if gated else ('gelu_' if gelu else '')}{_suffix(a.dtype)}"
+    name = f"tkb_moe_gemm_{'gated_' if gated else (act + '_' if act else '')}{_suffix(a.dtype)}"
     extra = (_ptr(pair_scale),) if gated else ()
     _check(_fn(_libs.get("moe.cu"), name)(_ptr(a), c_int(a.stride(0)), _ptr(w), _ptr(out), c_int(out.stride(0)),
                                           _ptr(offsets), _ptr(order), c_int(top), c_int(out.shape[0]), c_int(E), c_int(N),
@@ -1164,6 +1198,24 @@ def scaled_norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, scal
     _check(_fn(_libs.get("post_norm.cu"), f"tkb_scaled_norm_add_{suf}")(
         _ptr(x), _ptr(y), c_int(n_slices), ctypes.c_longlong(rows * H), _ptr(bias), _ptr(weight), _ptr(scale), c_float(mult),
         c_float(eps), _ptr(h_out), c_int(rows), c_int(H), _stream()), "scaled_norm_add")
+
+
+def norm_add_norm(x: torch.Tensor, y: torch.Tensor, w1: torch.Tensor, eps1: float, w2: torch.Tensor, eps2: float,
+                  out: torch.Tensor) -> None:
+    """x += w1 * N(y) in place, then out = w2 * N(x): the norm on a sublayer's output, the residual sum and the next
+    sublayer's norm in one pass.  x float32 [rows, H]; y float32 [rows, H] or the slices [slices, rows, H] of a split
+    product, added in slice order; out in the activation type."""
+    _need_cuda(x, y, w1, w2, out)
+    rows, H = x.shape
+    n_slices = y.shape[0] if y.dim() == 3 else 1
+    _need(x.dtype == torch.float32 and x.is_contiguous() and y.dtype == torch.float32 and y.is_contiguous()
+          and tuple(y.shape[-2:]) == (rows, H), "norm_add_norm: x and y contiguous float32 of one shape")
+    for w in (w1, w2):
+        _need(w.dtype == torch.float32 and w.is_contiguous() and w.numel() == H, "norm_add_norm: norm weights float32 [H]")
+    _need(out.shape == x.shape and out.is_contiguous(), "norm_add_norm: out of x's shape")
+    _check(_fn(_libs.get("post_norm.cu"), f"tkb_norm_add_norm_{_suffix(out.dtype)}")(
+        _ptr(x), _ptr(y), c_int(n_slices), ctypes.c_longlong(rows * H), _ptr(w1), c_float(eps1), _ptr(w2), c_float(eps2),
+        _ptr(out), c_int(rows), c_int(H), _stream()), "norm_add_norm")
 
 
 def linear_out_f32(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor | None) -> torch.Tensor:
@@ -1507,9 +1559,11 @@ def silu_cols(x: torch.Tensor, ncols: int, defines: dict) -> None:
 
 # ---------------------------------------------------------------------------------------------
 # Attention with a score cap and a sink, keys and values of different sizes (csrc/attention_sink.cu)
-def sink_attention_defines(dim: int, vdim: int, sigmoid: bool = False, maps: int = 1, distance: bool = False) -> dict:
+def sink_attention_defines(dim: int, vdim: int, sigmoid: bool = False, maps: int = 1, distance: bool = False,
+                           taps: int = 0) -> dict:
     """``sigmoid``: the build whose weights are sigmoid(score), not a softmax.  ``maps``: attention maps a head (each
-    with query and key vectors of its own, over the same values).  ``distance``: the build with a bias by distance."""
+    with query and key vectors of its own, over the same values).  ``distance``: the build with a bias by distance.
+    ``taps``: the build with a convolution of so many taps behind the projections."""
     _need(0 < dim <= 512 and 0 < vdim <= 512, f"sink attention: head sizes up to 512, not {dim} / {vdim}")
     _need(1 <= maps <= 4, f"sink attention: one to four maps a head, not {maps}")
     d = dict(TKB_QK=dim, TKB_VD=vdim)
@@ -1519,7 +1573,61 @@ def sink_attention_defines(dim: int, vdim: int, sigmoid: bool = False, maps: int
         d["TKB_MAPS"] = maps
     if distance:
         d["TKB_DIST"] = 1
+    if taps:
+        _need(0 < taps <= 16, f"sink attention: one to sixteen taps, not {taps}")
+        d["TKB_TAPS"] = taps
     return d
+
+
+def _sink_lib(dim, vdim, sigmoid=False, maps=1, distance=False, taps=0):
+    return _libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, distance, taps))
+
+
+def _sink_prep_checks(what: str, qkv, q_out, cache, n_heads, n_kv_heads, dim, vdim, page_size, maps, columns, norm_w,
+                      norm_w_shape, rot_freq, rot_dims) -> None:
+    T = qkv.shape[0]
+    _need(norm_w is None or (norm_w.dtype == torch.float32 and norm_w.is_contiguous() and tuple(norm_w.shape) == norm_w_shape),
+          f"{what}: norm weights float32 {list(norm_w_shape)}")
+    _need(rot_freq is None or (rot_freq.dtype == torch.float64 and rot_freq.is_contiguous() and rot_dims % 2 == 0
+                               and 0 < rot_dims <= dim and rot_freq.numel() == rot_dims // 2),
+          f"{what}: float64 [rot_dims / 2] frequencies")
+    _need(qkv.dtype == torch.float32 and qkv.stride(1) == 1 and qkv.shape[1] >= columns, f"{what}: float32 projections")
+    _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, n_heads * maps * dim) and q_out.dtype == cache.dtype, f"{what}: q_out")
+    _need(cache.is_contiguous() and tuple(cache.shape[1:]) == (n_kv_heads, page_size, maps * dim + vdim), f"{what}: cache rows")
+
+
+def sink_attn_conv_prep(qkv: torch.Tensor, taps: torch.Tensor, state: torch.Tensor | None, unit_norm: bool, eps: float,
+                        q_out: torch.Tensor, cache: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor,
+                        seq_slot: torch.Tensor, seq_q_start: torch.Tensor, seq_q_len: torch.Tensor, n_seqs: int,
+                        portions: bool, page_indptr: torch.Tensor, page_ids: torch.Tensor, n_heads: int, n_kv_heads: int,
+                        dim: int, vdim: int, page_size: int, write_cache: bool, write_state: bool, status: torch.Tensor,
+                        norm_w: torch.Tensor | None = None, rot_freq: torch.Tensor | None = None, rot_dims: int = 0,
+                        rot_pairs: bool = False, maps: int = 1, own_kv: bool = True, sigmoid: bool = False,
+                        distance: bool = False) -> None:
+    """``sink_attn_prep`` behind a causal convolution a channel of q, k and v: taps float32 [columns, n], the last one
+    meeting the token's own value; state float32 [slots, >= (n - 1) * columns], a request's last n - 1 projected rows,
+    which this moves on (None with one tap).  No biases.  ``portions``: whether the step can hold requests with several
+    tokens.  ``own_kv`` False: the projections hold q alone, nothing is cached."""
+    _need_cuda(qkv, taps, state, q_out, cache, positions, token_seq, seq_slot, seq_q_start, seq_q_len, page_indptr, page_ids,
+               status, norm_w, rot_freq)
+    T = qkv.shape[0]
+    C = (n_heads + (n_kv_heads if own_kv else 0)) * maps * dim + (n_kv_heads * vdim if own_kv else 0)
+    n = taps.shape[1]
+    _sink_prep_checks("sink_attn_conv_prep", qkv, q_out, cache, n_heads, n_kv_heads, dim, vdim, page_size, maps, C, norm_w,
+                      (2, dim), rot_freq, rot_dims)
+    _need(taps.dtype == torch.float32 and taps.is_contiguous() and taps.shape[0] == C, "sink_attn_conv_prep: taps float32 [columns, n]")
+    _need(n == 1 or (state is not None and state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+                     and state.shape[1] >= (n - 1) * C), "sink_attn_conv_prep: state float32 [slots, (n - 1) * columns]")
+    for t, k in ((positions, T), (token_seq, T), (seq_slot, n_seqs), (seq_q_start, n_seqs), (seq_q_len, n_seqs)):
+        _need(t.dtype == torch.int32 and t.numel() >= k, "sink_attn_conv_prep: int32 step arrays")
+    _check(_fn(_sink_lib(dim, vdim, sigmoid, maps, distance, n), f"tkb_sink_attn_conv_prep_{_suffix(cache.dtype)}")(
+        _ptr(qkv), c_int(qkv.stride(0)), _ptr(taps), _ptr(state if n > 1 else None),
+        ctypes.c_longlong(state.stride(0) if n > 1 else 0), c_int(1 if unit_norm else 0), c_float(eps), _ptr(q_out), _ptr(cache),
+        _ptr(positions), _ptr(token_seq), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(page_indptr),
+        _ptr(page_ids), c_int(T), c_int(n_seqs), c_int(1 if portions else 0), c_int(n_heads), c_int(n_kv_heads),
+        c_int(page_size), c_int(cache.shape[0]), c_int(1 if write_cache else 0), c_int(1 if write_state else 0), _ptr(status),
+        _ptr(norm_w), _ptr(rot_freq), c_int(rot_dims if rot_freq is not None else 0), c_int(1 if rot_pairs else 0),
+        c_int(1 if own_kv else 0), _stream()), "sink_attn_conv_prep")
 
 
 def sink_attn_prep(qkv: torch.Tensor, bias: torch.Tensor | None, unit_norm: bool, eps: float, q_out: torch.Tensor,
@@ -1527,33 +1635,32 @@ def sink_attn_prep(qkv: torch.Tensor, bias: torch.Tensor | None, unit_norm: bool
                    page_ids: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, vdim: int, page_size: int,
                    write_cache: bool, status: torch.Tensor, norm_w: torch.Tensor | None = None,
                    rot_freq: torch.Tensor | None = None, rot_dims: int = 0, rot_pairs: bool = False,
-                   values_are_keys: bool = False, sigmoid: bool = False, maps: int = 1, distance: bool = False) -> None:
+                   values_are_keys: bool = False, sigmoid: bool = False, maps: int = 1, distance: bool = False,
+                   whole_norm: bool = False, own_kv: bool = True, taps: int = 0) -> None:
     """qkv float32 [T, heads*maps*dim | kv heads*maps*dim | kv heads*vdim | anything else] -> (+ bias, q and k vectors
     divided by their root mean square) q_out [T, heads*maps*dim] and the tokens' [k of every map | v] rows in cache
     [pages, kv heads, page_size, maps*dim + vdim].
     ``norm_w`` float32 [2, dim]: weights of the q heads' and the k heads' norm.  ``rot_freq`` float64 [rot_dims / 2]:
     q and k are rotated by position on their first ``rot_dims`` channels (``rot_pairs``: channel 2i with 2i + 1, else
     i with i + rot_dims / 2).  ``values_are_keys``: the projections hold no v; a token's value is its key as projected
-    (before norm and rotation).  ``sigmoid``, ``distance``: the kernel build that the attention itself uses."""
+    (before norm and rotation).  ``sigmoid``, ``distance``, ``taps``: the kernel build that the attention itself uses.
+    ``whole_norm``: q is divided by one root mean square over all its vectors, and so is k; ``norm_w`` then holds a weight
+    for every column of q and k.  ``own_kv`` False: the projections hold q alone, nothing is cached (the layer reads rows
+    that another layer wrote)."""
     _need_cuda(qkv, bias, q_out, cache, positions, token_seq, page_indptr, page_ids, status, norm_w, rot_freq)
     T = qkv.shape[0]
-    C = (n_heads + n_kv_heads) * maps * dim + (0 if values_are_keys else n_kv_heads * vdim)
+    QK = (n_heads + (n_kv_heads if own_kv else 0)) * maps * dim
+    C = QK + (0 if values_are_keys or not own_kv else n_kv_heads * vdim)
     _need(not values_are_keys or (dim == vdim and maps == 1), "sink_attn_prep: values that are the keys have the keys' size")
-    _need(norm_w is None or (norm_w.dtype == torch.float32 and norm_w.is_contiguous() and tuple(norm_w.shape) == (2, dim)),
-          "sink_attn_prep: norm weights float32 [2, dim]")
-    _need(rot_freq is None or (rot_freq.dtype == torch.float64 and rot_freq.is_contiguous() and rot_dims % 2 == 0
-                               and 0 < rot_dims <= dim and rot_freq.numel() == rot_dims // 2),
-          "sink_attn_prep: float64 [rot_dims / 2] frequencies")
-    _need(qkv.dtype == torch.float32 and qkv.stride(1) == 1 and qkv.shape[1] >= C, "sink_attn_prep: float32 projections")
+    _sink_prep_checks("sink_attn_prep", qkv, q_out, cache, n_heads, n_kv_heads, dim, vdim, page_size, maps, C, norm_w,
+                      (QK,) if whole_norm else (2, dim), rot_freq, rot_dims)
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == C), "sink_attn_prep: bias float32")
-    _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, n_heads * maps * dim) and q_out.dtype == cache.dtype, "sink_attn_prep: q_out")
-    _need(cache.is_contiguous() and tuple(cache.shape[1:]) == (n_kv_heads, page_size, maps * dim + vdim), "sink_attn_prep: cache rows")
-    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, distance)), f"tkb_sink_attn_prep_{_suffix(cache.dtype)}")(
-        _ptr(qkv), c_int(qkv.stride(0)), _ptr(bias), c_int(1 if unit_norm else 0), c_float(eps), _ptr(q_out), _ptr(cache),
+    _check(_fn(_sink_lib(dim, vdim, sigmoid, maps, distance, taps), f"tkb_sink_attn_prep_{_suffix(cache.dtype)}")(
+        _ptr(qkv), c_int(qkv.stride(0)), _ptr(bias), c_int(2 if whole_norm else (1 if unit_norm else 0)), c_float(eps), _ptr(q_out), _ptr(cache),
         _ptr(positions), _ptr(token_seq), _ptr(page_indptr), _ptr(page_ids), c_int(T), c_int(n_heads), c_int(n_kv_heads),
         c_int(page_size), c_int(cache.shape[0]), c_int(1 if write_cache else 0), _ptr(status), _ptr(norm_w), _ptr(rot_freq),
         c_int(rot_dims if rot_freq is not None else 0), c_int(1 if rot_pairs else 0), c_int(1 if values_are_keys else 0),
-        _stream()), "sink_attn_prep")
+        c_int(1 if own_kv else 0), _stream()), "sink_attn_prep")
 
 
 def _row_stride(t: torch.Tensor) -> int:
@@ -1573,20 +1680,29 @@ def _sink_out_ok(out: torch.Tensor, rows: int, n_heads: int, vdim: int, maps: in
             and out.dtype == (act if maps == 1 else torch.float32))
 
 
+def _sink_gate(gate: torch.Tensor | None, tokens: int, n_heads: int, maps: int, what: str) -> tuple:
+    """The gate's pointer and row stride as kernel arguments."""
+    _need_cuda(gate)
+    _need(gate is None or (maps == 1 and gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1
+                           and gate.shape[0] >= tokens and gate.shape[1] == n_heads), f"{what}: gate logits float32 [tokens, heads]")
+    return _ptr(gate), c_int(_row_stride(gate) if gate is not None else 0)
+
+
 def attn_sink(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, token_seq: torch.Tensor, positions: torch.Tensor,
               page_indptr: torch.Tensor, page_ids: torch.Tensor, rows: torch.Tensor | None, n_rows: int,
               sinks: torch.Tensor | None, n_heads: int, n_kv_heads: int, dim: int, vdim: int, page_size: int,
               scale: float, softcap: float | None, window: int | None, status: torch.Tensor,
               head_scale: torch.Tensor | None = None, head_bias: torch.Tensor | None = None, sigmoid: bool = False,
               maps: int = 1, keep_first: int = 0, chunk: int | None = None, head_slope: torch.Tensor | None = None,
-              out_scale: float = 1.0) -> None:
+              out_scale: float = 1.0, gate: torch.Tensor | None = None, taps: int = 0) -> None:
     """Attention of ``n_rows`` tokens (``rows`` names them; None: all) over their requests' cached [k | v] rows.
     ``head_scale`` / ``head_bias`` float32 [heads]: a factor on a head's scale, a number added to its scores.
     ``sigmoid``: weights sigmoid(score) instead of a softmax (no sink).  ``maps`` > 1: so many attention maps a head,
     each a softmax of its own; ``out`` then is float32 [rows, heads * maps * vdim].  ``keep_first``: with a window, the
     request's first so many positions stay visible.  ``chunk``: a query sees the keys of its own chunk of so many positions
     only.  ``head_slope`` float32 [heads]: a slope times the distance comes off a head's scores.  ``out_scale`` multiplies
-    the result; ``out`` may be a column slice of a wider tensor."""
+    the result; ``out`` may be a column slice of a wider tensor.  ``gate`` float32 [tokens, heads] (one map; a column slice
+    will do): head h's result of token t counts sigmoid(gate[t, h]) times.  ``taps``: the kernel build."""
     _need_cuda(q, out, cache, token_seq, positions, page_indptr, page_ids, rows, sinks, status, head_scale, head_bias, head_slope)
     _head_vectors(n_heads * maps, "attn_sink", head_scale, head_bias, head_slope)
     _need(not (sigmoid and sinks is not None), "attn_sink: the sigmoid form has no sink")
@@ -1594,12 +1710,13 @@ def attn_sink(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, token_seq
           and _sink_out_ok(out, n_rows, n_heads, vdim, maps, cache.dtype), "attn_sink: q and out")
     _need(cache.is_contiguous() and tuple(cache.shape[1:]) == (n_kv_heads, page_size, maps * dim + vdim), "attn_sink: cache rows")
     _need(sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == n_heads * maps), "attn_sink: sinks float32 [heads]")
-    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, head_slope is not None)), f"tkb_attn_sink_simt_{_suffix(cache.dtype)}")(
+    gate_args = _sink_gate(gate, q.shape[0], n_heads, maps, "attn_sink")
+    _check(_fn(_sink_lib(dim, vdim, sigmoid, maps, head_slope is not None, taps), f"tkb_attn_sink_simt_{_suffix(cache.dtype)}")(
         _ptr(q), _ptr(out), _ptr(cache), _ptr(token_seq), _ptr(positions), _ptr(page_indptr), _ptr(page_ids), _ptr(rows),
         c_int(n_rows), _ptr(sinks), c_int(n_heads), c_int(n_kv_heads), c_int(page_size), c_float(scale),
         c_float(softcap or 0.0), c_int(window or 0), c_int(keep_first if window else 0), c_int(chunk or 0),
         c_int(cache.shape[0]), _ptr(status), _ptr(head_scale), _ptr(head_bias), _ptr(head_slope), c_int(_row_stride(out)),
-        c_float(out_scale), _stream()), "attn_sink")
+        c_float(out_scale), *gate_args, _stream()), "attn_sink")
 
 
 def can_use_attn_sink_tc(dtype: torch.dtype, dim: int, vdim: int, maps: int = 1) -> bool:
@@ -1614,10 +1731,11 @@ def attn_sink_tc(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, seq_q_
                  softcap: float | None, window: int | None, status: torch.Tensor, portions: bool = True,
                  singles: bool = True, head_scale: torch.Tensor | None = None, head_bias: torch.Tensor | None = None,
                  sigmoid: bool = False, maps: int = 1, keep_first: int = 0, chunk: int | None = None,
-                 head_slope: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
+                 head_slope: torch.Tensor | None = None, out_scale: float = 1.0, gate: torch.Tensor | None = None,
+                 taps: int = 0) -> None:
     """Attention of every token of the step on the tensor cores (bfloat16): out [T, heads * vdim] (``maps`` > 1: float32
     [T, heads * maps * vdim]).  ``portions`` / ``singles``: whether the step can hold requests with several tokens /
-    with one (a kernel each).  ``keep_first``, ``chunk``, ``head_slope``, ``out_scale``: as in ``attn_sink``."""
+    with one (a kernel each).  ``keep_first``, ``chunk``, ``head_slope``, ``out_scale``, ``gate``, ``taps``: as in ``attn_sink``."""
     _need_cuda(q, out, cache, seq_q_start, seq_q_len, seq_kv_len, page_indptr, page_ids, sinks, status, head_scale, head_bias, head_slope)
     _head_vectors(n_heads * maps, "attn_sink_tc", head_scale, head_bias, head_slope)
     _need(not (sigmoid and sinks is not None), "attn_sink_tc: the sigmoid form has no sink")
@@ -1639,12 +1757,13 @@ def attn_sink_tc(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, seq_q_
             splits = min(splits, max(1, (min(w for w in (window, chunk) if w) + 63) // 64))
         if splits > 1:
             part = torch.empty((n_seqs * n_heads * maps * splits * (vdim + 2),), dtype=torch.float32, device=q.device)
-    _check(_fn(_libs.get("attention_sink.cu", **sink_attention_defines(dim, vdim, sigmoid, maps, head_slope is not None)), "tkb_attn_sink_tc_bf16")(
+    gate_args = _sink_gate(gate, T, n_heads, maps, "attn_sink_tc")
+    _check(_fn(_sink_lib(dim, vdim, sigmoid, maps, head_slope is not None, taps), "tkb_attn_sink_tc_bf16")(
         _ptr(q), _ptr(out), _ptr(cache), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(page_indptr),
         _ptr(page_ids), c_int(T), c_int(n_seqs), c_int(1 if portions else 0), c_int(1 if singles else 0), _ptr(sinks),
         c_int(n_heads), c_int(n_kv_heads), c_int(page_size), c_float(scale), c_float(softcap or 0.0), c_int(window or 0),
         c_int(keep_first if window else 0), c_int(chunk or 0), c_int(cache.shape[0]), _ptr(status), _ptr(part), c_int(splits),
-        _ptr(head_scale), _ptr(head_bias), _ptr(head_slope), c_int(_row_stride(out)), c_float(out_scale), _stream()), "attn_sink_tc")
+        _ptr(head_scale), _ptr(head_bias), _ptr(head_slope), c_int(_row_stride(out)), c_float(out_scale), *gate_args, _stream()), "attn_sink_tc")
 
 
 def diff_combine(a: torch.Tensor, lam: torch.Tensor, eps: float, mult: float, gate: torch.Tensor | None, gate_off: int,

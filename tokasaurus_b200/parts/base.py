@@ -40,6 +40,8 @@ class WeightSpec:
     keep_32bit: bool = False
     # A tensor that a checkpoint may lack: the part then finds no entry under its name and does without.
     optional: bool = False
+    # A table's entries lie below this number and differ within a row (0: any integers).
+    below: int = 0
 
 
 @dataclass(frozen=True)
@@ -182,20 +184,29 @@ class ResidualStream:
     """The running sum of a token's representation, held in float32, plus one pending
     update in the engine's dtype that the next norm adds before it normalises (so the add
     costs no extra pass over memory).  The update may also be float32 slices of a split product, or (norms that
-    take them) a pair of float32 updates, of the two sublayers of a block that read one norm.  ``h``: the same rows as ``x`` in the activation type, if the kernel that made
+    take them) a pair of float32 updates, of the two sublayers of a block that read one norm.  ``delta_norm``: an RMS norm
+    through which the update goes before it is added (a block with norms on its sublayers' outputs as well; only
+    ``parts.norm.RMSNorm`` takes such a stream further).  ``h``: the same rows as ``x`` in the activation type, if the kernel that made
     ``x`` wrote them too (blocks whose sublayers read the stream itself)."""
 
-    __slots__ = ("x", "delta", "h")
+    __slots__ = ("x", "delta", "h", "delta_norm")
 
     def __init__(self, x: "torch.Tensor", delta: "torch.Tensor | None" = None, h: "torch.Tensor | None" = None):
         self.x = x
         self.delta = delta
         self.h = h
+        self.delta_norm = None
 
     def settled(self) -> "torch.Tensor":
         """A copy of the rows with the pending update added (for looking at a model layer by layer)."""
+        import torch
+
         x = self.x.clone()
         for d in (self.delta if isinstance(self.delta, (tuple, list)) else (self.delta,)):
             if d is not None:
-                x += d.sum(0) if d.dim() == 3 else d
+                d = d.sum(0) if d.dim() == 3 else d
+                if self.delta_norm is not None:
+                    n = self.delta_norm
+                    d = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + n.eps) * n.weight
+                x += d
         return x

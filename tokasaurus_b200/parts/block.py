@@ -27,6 +27,13 @@ def _mix(mixer: Mixer, ctx, h, cache, out_rows, state: dict | None):
     return mixer.forward(ctx, h, cache, out_rows)
 
 
+def _feed(ffn: FeedForward, ctx, h, out_rows):
+    """``ffn.forward``; a feed-forward that goes by token ids is told which tokens its rows belong to (None: all)."""
+    if getattr(ffn, "by_token", False):
+        return ffn.forward(ctx, h, rows=out_rows)
+    return ffn.forward(ctx, h)
+
+
 class PreNormBlock(Part):
     def __init__(self, mixer_norm: Norm, mixer: Mixer, ffn_norm: Norm | None, ffn: FeedForward | None,
                  mixer_stage: InputStage | None = None, ffn_stage: InputStage | None = None):
@@ -93,7 +100,7 @@ class PreNormBlock(Part):
             hc = torch.empty((out_rows.numel(), h.shape[1]), dtype=h.dtype, device=h.device)
             ops.gather_rows(h, out_rows, hc)
             h = hc
-        stream.delta = self.ffn.forward(ctx, h)
+        stream.delta = _feed(self.ffn, ctx, h, out_rows)
         return stream
 
     @staticmethod
@@ -142,7 +149,55 @@ class ParallelBlock(Part):
             hc = torch.empty((out_rows.numel(), h.shape[1]), dtype=h.dtype, device=h.device)
             ops.gather_rows(h, out_rows, hc)
             h = hc
-        stream.delta = (mixed, self.ffn.forward(ctx, h))
+        stream.delta = (mixed, _feed(self.ffn, ctx, h, out_rows))
+        return stream
+
+
+class SandwichNormBlock(Part):
+    """A block with a norm ahead of each sublayer and another on its output:
+
+        x <- x + norm1b(mixer(norm1(x))),      x <- x + norm2b(ffn(norm2(x)))
+
+    The norms are RMS norms (``parts.norm.RMSNorm``).  A sublayer leaves its output pending together with its output norm
+    (``ResidualStream.delta_norm``); the next norm, which may be the next block's or the head's, does both norms and the
+    sum between them in one pass.  ``ffn=None``: the block is its mixer alone.  A feed-forward that goes by token ids
+    (``by_token``) is told which tokens its rows belong to."""
+
+    def __init__(self, mixer_norm, mixer: Mixer, mixer_out_norm, ffn_norm=None, ffn: FeedForward | None = None,
+                 ffn_out_norm=None):
+        if (ffn is None) != (ffn_norm is None) or (ffn is None) != (ffn_out_norm is None):
+            raise ValueError("a block has a feed-forward and its two norms, or none of them")
+        self.mixer_norm, self.mixer, self.mixer_out_norm = mixer_norm, mixer, mixer_out_norm
+        self.ffn_norm, self.ffn, self.ffn_out_norm = ffn_norm, ffn, ffn_out_norm
+
+    def parts(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.ffn_norm, self.ffn,
+                                 self.ffn_out_norm) if p is not None)
+
+    def weight_specs(self):
+        return tuple(s for p in self.parts() for s in p.weight_specs())
+
+    def kernel_modules(self, dtype):
+        return (("post_norm.cu", None),) + tuple(m for p in self.parts() for m in p.kernel_modules(dtype))
+
+    def bind(self, weights, rt) -> None:
+        for p in self.parts():
+            p.bind(weights, rt)
+
+    def state_needs(self) -> dict:
+        return _side_needs(self.mixer)
+
+    def forward(self, ctx, stream: ResidualStream, cache, out_rows=None, stage_state=None) -> ResidualStream:
+        h = self.mixer_norm.forward(ctx, stream)
+        if out_rows is not None:
+            stream = PreNormBlock._cut(stream, out_rows)
+        stream.delta = _mix(self.mixer, ctx, h, cache, out_rows, stage_state)
+        stream.delta_norm = self.mixer_out_norm
+        if self.ffn is None:
+            return stream
+        h = self.ffn_norm.forward(ctx, stream)
+        stream.delta = _feed(self.ffn, ctx, h, out_rows)
+        stream.delta_norm = self.ffn_out_norm
         return stream
 
 
@@ -207,7 +262,7 @@ class OutputNormBlock(Part):
             stream = PreNormBlock._cut(stream, out_rows)
         self._add(stream, y, self.mixer_norm, self.scales[0], getattr(self.mixer, "out_bias", None))
         if self.ffn is not None:
-            self._add(stream, self.ffn.forward(ctx, self._input(stream)), self.ffn_norm, self.scales[1])
+            self._add(stream, _feed(self.ffn, ctx, self._input(stream), out_rows), self.ffn_norm, self.scales[1])
         return stream
 
 
@@ -262,7 +317,7 @@ class PostNormBlock(Part):
             stream = PreNormBlock._cut(stream, out_rows)
         stream.h = self.mixer_norm.apply_sum(stream.x, y, self.alpha)
         if self.ffn is not None:
-            stream.h = self.ffn_norm.apply_sum(stream.x, self.ffn.forward(ctx, self._input(stream)), self.alpha)
+            stream.h = self.ffn_norm.apply_sum(stream.x, _feed(self.ffn, ctx, self._input(stream), out_rows), self.alpha)
         elif self.ffn_norm is not None and self.ffn_norm.weight is not None:
             stream.h = self.ffn_norm.apply_sum(stream.x, None, self.alpha)
         if self.side is not None:

@@ -36,7 +36,7 @@ class DifferentialAttention(SinkAttention):
                          extra_names=((gate_name, n_heads),) if gate_name is not None else ())
         self.diff = float(diff)
         self.lambda_names = tuple(lambda_names)
-        self.gated = gate_name is not None
+        self.diff_gated = gate_name is not None
         self.lam: torch.Tensor | None = None
 
     def weight_specs(self):
@@ -49,6 +49,6 @@ class DifferentialAttention(SinkAttention):
 
     def _combine(self, ctx, attn, qkv, out_rows):
         out = torch.empty((attn.shape[0], self.n_heads * self.vdim), dtype=self.w_o.dtype, device=attn.device)
-        ops.diff_combine(attn, self.lam, self.norm_eps, 1.0 - self.diff, qkv if self.gated else None, self.extra_off,
+        ops.diff_combine(attn, self.lam, self.norm_eps, 1.0 - self.diff, qkv if self.diff_gated else None, self.extra_off,
                          out_rows, out, self.n_heads, self.dim, self.vdim)
         return out

@@ -43,9 +43,10 @@ class TokenEmbedding(Part):
 
 class OutputHead(Part):
     """``weight_name`` may be the embedding's tensor (tied weights): the loader hands the same
-    storage to both parts."""
+    storage to both parts.  ``softcap``: the logits become softcap * tanh(logits / softcap)."""
 
-    def __init__(self, vocab: int, width: int, norm: Norm, weight_name: str):
+    def __init__(self, vocab: int, width: int, norm: Norm, weight_name: str, softcap: float | None = None):
+        self.softcap = float(softcap) if softcap else None
         self.vocab = vocab
         self.width = width
         self.norm = norm
@@ -64,4 +65,7 @@ class OutputHead(Part):
 
     def forward(self, ctx, stream: ResidualStream) -> torch.Tensor:
         h = self.norm.forward(ctx, stream)
-        return ops.linear(h, self.weight, out_dtype=torch.float32)
+        logits = ops.linear(h, self.weight, out_dtype=torch.float32)
+        if self.softcap is not None:
+            ops.soft_cap(logits, self.softcap)
+        return logits

@@ -74,13 +74,16 @@ class GatedMLP(FeedForward):
         return ops.linear(act, self.w_down, out_dtype=torch.float32 if self.out_f32 else None)
 
 
-class GeluMLP(FeedForward):
-    """``down(gelu(up(h)))`` with the exact (erf) GELU, no gate, no biases.  Many rows in bfloat16: the GELU is the
-    epilogue of the tcgen05 up product; few rows: the K-split product's float32 slices go through one activation kernel;
-    float32: the activation kernel behind the float32 product.  The update leaves as float32 rows or slices."""
+class UngatedMLP(FeedForward):
+    """``down(act(up(h)))`` without a gate and without biases; ``activation`` "gelu" (the exact, erf form) or "relu2" (the
+    square of relu).  Many rows in bfloat16: the activation is the epilogue of the tcgen05 up product; few rows: the
+    K-split product's float32 slices go through one activation kernel; float32: the activation kernel behind the float32
+    product.  The update leaves as float32 rows or slices."""
 
-    def __init__(self, width: int, inner: int, up_name: str, down_name: str):
-        self.width, self.inner = width, inner
+    def __init__(self, width: int, inner: int, up_name: str, down_name: str, activation: str):
+        if activation not in ops.UNGATED_ACTS:
+            raise ValueError(f"an ungated activation is one of {sorted(ops.UNGATED_ACTS)}, not {activation!r}")
+        self.width, self.inner, self.activation = width, inner, activation
         self.names = (up_name, down_name)
 
     def weight_specs(self):
@@ -97,12 +100,26 @@ class GeluMLP(FeedForward):
         if h.shape[0] >= ops.TCGEN05_M_MIN and ops.can_use_tcgen05(h, self.w_up):
             if status is None:
                 status = torch.zeros(1, dtype=torch.int32, device=h.device)
-            act = ops.gemm_tcgen05(h, self.w_up, status, gelu=True)
+            act = ops.gemm_tcgen05(h, self.w_up, status, act=self.activation)
         else:
             z = ops.linear_out_f32(h, self.w_up, status)
             act = torch.empty((h.shape[0], self.inner), dtype=h.dtype, device=h.device)
-            ops.gelu_rows(z, act)
+            ops.act_rows(z, act, self.activation)
         return ops.linear_out_f32(act, self.w_down, status)
+
+
+class GeluMLP(UngatedMLP):
+    """``down(gelu(up(h)))`` with the exact (erf) GELU."""
+
+    def __init__(self, width: int, inner: int, up_name: str, down_name: str):
+        super().__init__(width, inner, up_name, down_name, "gelu")
+
+
+class SquaredReluMLP(UngatedMLP):
+    """``down(relu(up(h))^2)``."""
+
+    def __init__(self, width: int, inner: int, up_name: str, down_name: str):
+        super().__init__(width, inner, up_name, down_name, "relu2")
 
 
 class ClampedGLU(FeedForward):
@@ -187,8 +204,8 @@ class RoutedExperts(FeedForward):
     s = sigmoid(logits); the choice goes by s + correction (a learned vector that takes no part in the weights), among
     the experts of the best ``keep`` of ``groups`` equal groups of neighbours only (a group scores the sum of its two
     largest choice scores); the weights are the chosen experts' s over their sum, times ``scale``.
-    ``expert="gelu"``: an expert is ``down(gelu(up h))`` with the exact GELU and no gate; ``expert_names(e)`` then gives
-    (up, down).  ``out_dtype`` float32: the weighted sum leaves as float32 rows (for a norm that reads it).
+    ``expert="gelu"``: an expert is ``down(gelu(up h))`` with the exact GELU and no gate (``"relu2"``: the square of relu in
+    its place); ``expert_names(e)`` then gives (up, down).  ``out_dtype`` float32: the weighted sum leaves as float32 rows (for a norm that reads it).
     ``scored`` with ``renormalize=False``: the chosen scores times ``scale`` as they are.
 
     ``weigh_input`` (SiLU-gated experts): a choice's weight multiplies what goes INTO the expert, the output is the plain
@@ -198,7 +215,10 @@ class RoutedExperts(FeedForward):
     the chosen experts' shares of the softmax over ALL experts, times ``scale``, not renormalised.
     ``expert="clamped"`` with ``clamp`` = (limit, alpha): an expert is ``down(g * sigmoid(alpha g) * (u + 1))`` with
     g = min(gate(h), limit), u = clamp(up(h), -limit, limit).  ``shared_gate_name``: a vector [1, width]; the shared
-    expert's output counts sigmoid(that vector . h) times, one number a token (float32)."""
+    expert's output counts sigmoid(that vector . h) times, one number a token (float32).
+
+    ``table_name``: no router.  An int32 table [vocab, top] gives each token id its experts, each of weight 1 / top; the
+    layer then asks for the tokens its rows belong to (``by_token``, ``forward(..., rows=)``)."""
 
     # (token, choice) pairs from which the gathered tcgen05 products are used (bfloat16).  Below, the few-rows kernel
     # fetches every chosen expert's weights once as well, but spends one multiply-add a row on every weight it
@@ -207,15 +227,21 @@ class RoutedExperts(FeedForward):
     # 1,024 x 4,096, four chosen: 8 pairs 117 against 118, 16 pairs 179 against 132, 96 pairs 366 against 219).
     TENSOR_CORE_PAIRS_MIN = 12
 
-    def __init__(self, width: int, inner: int, n_experts: int, top: int, router_name: str, router_bias_name: str | None,
+    def __init__(self, width: int, inner: int, n_experts: int, top: int, router_name: str | None, router_bias_name: str | None,
                  expert_names, shared: FeedForward | None = None, scored: dict | None = None, expert: str = "silu_gated",
                  out_dtype: torch.dtype | None = None, over_all: dict | None = None, clamp: tuple[float, float] | None = None,
-                 shared_gate_name: str | None = None, weigh_input: bool = False):
+                 shared_gate_name: str | None = None, weigh_input: bool = False, table_name: str | None = None,
+                 vocab: int = 0):
         """``expert_names(e)`` -> (gate, up, down) tensor names of expert e."""
         if not 0 < top <= n_experts:
             raise ValueError(f"top={top} of {n_experts} experts")
-        if expert not in ("silu_gated", "gelu", "clamped"):
-            raise ValueError(f"an expert is 'silu_gated', 'gelu' or 'clamped', not {expert!r}")
+        if expert not in ("silu_gated", "gelu", "relu2", "clamped"):
+            raise ValueError(f"an expert is 'silu_gated', 'gelu', 'relu2' or 'clamped', not {expert!r}")
+        if (router_name is None) == (table_name is None) or (table_name is not None and vocab <= 0):
+            raise ValueError("experts are chosen by a router or by a table of the vocabulary")
+        if table_name is not None and (scored is not None or over_all is not None or router_bias_name is not None or weigh_input):
+            raise ValueError("a table has no scores")
+        self.table_name, self.vocab, self.by_token = table_name, int(vocab), table_name is not None
         if (expert == "clamped") != (clamp is not None) or (clamp is not None and not clamp[0] > 0):
             raise ValueError("a clamped expert has a positive limit and a factor, other experts neither")
         if over_all is not None and scored is not None:
@@ -232,14 +258,18 @@ class RoutedExperts(FeedForward):
             g, keep = int(scored.get("groups", 1)), int(scored.get("keep", 1))
             if g <= 0 or n_experts % g or not 0 < keep <= g or top > keep * (n_experts // g):
                 raise ValueError(f"{n_experts} experts in {g} groups of which {keep} are kept, {top} chosen")
-        self.scored, self.gelu, self.out_dtype = scored, expert == "gelu", out_dtype
+        self.scored, self.out_dtype = scored, out_dtype
+        self.act = expert if expert in ops.UNGATED_ACTS else None  # None: a gated unit
         self.width, self.inner, self.n_experts, self.top = width, inner, n_experts, top
         self.router_name, self.router_bias_name = router_name, router_bias_name
         self.expert_names = [tuple(expert_names(e)) for e in range(n_experts)]
         self.shared = shared
 
     def weight_specs(self):
-        specs = [WeightSpec(self.router_name, (self.n_experts, self.width), role="vector")]
+        if self.table_name is not None:
+            specs = [WeightSpec(self.table_name, (self.vocab, self.top), role="table", below=self.n_experts)]
+        else:
+            specs = [WeightSpec(self.router_name, (self.n_experts, self.width), role="vector")]
         if self.router_bias_name is not None:
             specs.append(WeightSpec(self.router_bias_name, (self.n_experts,), role="vector"))
         if self.scored is not None and self.scored.get("correction") is not None:
@@ -257,7 +287,10 @@ class RoutedExperts(FeedForward):
         return (("moe.cu", None),) + tc + (tuple(self.shared.kernel_modules(dtype)) if self.shared is not None else ())
 
     def bind(self, weights, rt) -> None:
-        self.router_w = weights[self.router_name].contiguous()
+        self.router_w = weights[self.router_name].contiguous() if self.router_name is not None else None
+        self.table = weights[self.table_name].contiguous() if self.table_name is not None else None
+        if self.table is not None and (int(self.table.min()) < 0 or int(self.table.max()) >= self.n_experts):
+            raise ValueError(f"{self.table_name} names experts outside 0 .. {self.n_experts - 1}")
         # the shared expert's gate: a one-row product in float32, like the router's own
         self.shared_gate_w = (weights[self.shared_gate_name].float().view(1, self.width).contiguous()
                               if self.shared_gate_name is not None else None)
@@ -278,20 +311,27 @@ class RoutedExperts(FeedForward):
         self.w_gate_up_tc = None
         # (sizes below one tile of the kernel's TMA boxes stay with the other kernels)
         if rt.dtype == torch.bfloat16 and self.inner % 8 == 0 and self.width % 8 == 0 and self.inner >= 64 and self.width >= 128:
-            self.w_gate_up_tc = self.w_gate_up if self.gelu else torch.stack(
+            self.w_gate_up_tc = self.w_gate_up if self.act else torch.stack(
                 [ops.interleave_gate_up(weights[g], weights[u]) for g, u, _ in self.expert_names]).contiguous()
         if self.shared is not None:
             self.shared.bind(weights, rt)
 
-    def forward(self, ctx, h):
+    def forward(self, ctx, h, rows=None):
+        """``rows`` (only with a table): the tokens of the step that h's rows belong to (None: all, in order)."""
         T, dev = h.shape[0], h.device
         top, E = self.top, self.n_experts
         top_idx = torch.empty((T, top), dtype=torch.int32, device=dev)
         top_w = torch.empty((T, top), dtype=torch.float32, device=dev)
-        # rows of padding tokens (a step graph's) choose nothing; a cut-down set of rows has none
-        token_seq = ctx.token_seq if (ctx is not None and T == ctx.n_tokens) else None
-        ops.moe_route(h, self.router_w, self.router_b, token_seq, top, top_idx, top_w, self.route_args,
-                      over_all=self.over_all is not None, scale=float((self.over_all or {}).get("scale", 1.0)))
+        if self.table is not None:
+            if rows is None and T != ctx.n_tokens:
+                raise ValueError(f"{T} rows of {ctx.n_tokens} tokens: experts by token id need to know which")
+            ops.moe_table(self.table, E, ctx.token_ids, ctx.token_seq, ctx.seq_slot, ctx.last_token, rows, top_idx, top_w,
+                          ctx.status)
+        else:
+            # rows of padding tokens (a step graph's) choose nothing; a cut-down set of rows has none
+            token_seq = ctx.token_seq if (ctx is not None and T == ctx.n_tokens) else None
+            ops.moe_route(h, self.router_w, self.router_b, token_seq, top, top_idx, top_w, self.route_args,
+                          over_all=self.over_all is not None, scale=float((self.over_all or {}).get("scale", 1.0)))
         shared_gate = None
         if self.shared_gate_name is not None:
             shared_gate = torch.empty((T,), dtype=torch.float32, device=dev)
@@ -309,11 +349,11 @@ class RoutedExperts(FeedForward):
             src_token = torch.empty((n_tiles * tile,), dtype=torch.int32, device=dev)
             tile_group = torch.empty((n_tiles,), dtype=torch.int32, device=dev)
             ops.moe_order(top_idx, E, offsets, order, place_of, pad=tile, tile_group=tile_group, src_token=src_token)
-            rows = torch.empty((n_tiles * tile, self.width), dtype=h.dtype, device=dev)
+            placed = torch.empty((n_tiles * tile, self.width), dtype=h.dtype, device=dev)
             scale = torch.empty((n_tiles * tile,), dtype=torch.float32, device=dev) if self.weigh_input else None
-            ops.moe_gather(h, src_token, rows, order if self.weigh_input else None, top_w if self.weigh_input else None, scale)
+            ops.moe_gather(h, src_token, placed, order if self.weigh_input else None, top_w if self.weigh_input else None, scale)
             status = ctx.status if ctx is not None else torch.zeros(1, dtype=torch.int32, device=dev)
-            act = ops.gemm_tcgen05_grouped(rows, self.w_gate_up_tc, tile_group, status, gated=not self.gelu, gelu=self.gelu,
+            act = ops.gemm_tcgen05_grouped(placed, self.w_gate_up_tc, tile_group, status, gated=self.act is None, act=self.act,
                                            clamp=self.clamp, row_scale=scale)
             y = ops.gemm_tcgen05_grouped(act, self.w_down, tile_group, status)
             ops.moe_combine(y, place_of, top_w, shared, out, shared_gate, weigh=not self.weigh_input)
@@ -321,7 +361,7 @@ class RoutedExperts(FeedForward):
         order = torch.empty((T * top,), dtype=torch.int32, device=dev)
         ops.moe_order(top_idx, E, offsets, order, place_of)
         act = torch.empty((T * top, self.inner), dtype=h.dtype, device=dev)
-        ops.moe_gemm(h, self.w_gate_up, act, offsets, order, top, gated=not self.gelu, gelu=self.gelu, clamp=self.clamp,
+        ops.moe_gemm(h, self.w_gate_up, act, offsets, order, top, gated=self.act is None, act=self.act, clamp=self.clamp,
                      pair_scale=top_w if self.weigh_input else None)
         y = torch.empty((T * top, self.width), dtype=torch.float32, device=dev)
         ops.moe_gemm(act, self.w_down, y, offsets, None, top, gated=False)

@@ -38,7 +38,13 @@ class RMSNorm(Norm):
         return out
 
     def forward(self, ctx, stream: ResidualStream):
-        out = self._run(stream.x, stream.delta)
+        if stream.delta_norm is not None:  # the pending update is a sublayer's output that is normed on its way in
+            first = stream.delta_norm
+            out = torch.empty(stream.x.shape, dtype=self.out_dtype, device=stream.x.device)
+            ops.norm_add_norm(stream.x, stream.delta, first.weight, first.eps, self.weight, self.eps, out)
+            stream.delta_norm = None
+        else:
+            out = self._run(stream.x, stream.delta)
         stream.delta = None
         return out
 

@@ -63,13 +63,18 @@ class RotaryEncoding(PositionEncoding):
 
     def inv_freq64(self) -> torch.Tensor:
         """float64 [rotary_dim / 2] ``theta^(-2j / rotary_dim)``, on the CPU, for kernels that form their angles in
-        float64 (plain frequencies, or yarn's blend of scaled and unscaled ones)."""
-        if self.scaling_type not in ("default", "yarn"):
-            raise ValueError("float64 frequencies exist for the plain and the yarn rotary encoding")
+        float64, scaled as the encoding says."""
         d = self.rotary_dim
         f = self.theta ** (-torch.arange(0, d, 2, dtype=torch.float64) / d)
         if self.scaling_type == "default":
             return f
+        if self.scaling_type == "llama3":
+            orig, low, high = float(self.original_max_position_embeddings), self.low_freq_factor, self.high_freq_factor
+            wavelen = 2.0 * math.pi / f
+            # (equal factors: nothing lies between the two lengths)
+            smooth = (orig / wavelen - low) / (high - low) if high != low else torch.ones_like(f)
+            blend = (1.0 - smooth) * f / self.factor + smooth * f
+            return torch.where(wavelen < orig / high, f, torch.where(wavelen > orig / low, f / self.factor, blend))
         orig = float(self.original_max_position_embeddings)
 
         def turns(t: float) -> float:

@@ -34,6 +34,16 @@ their float32 results are the trailing columns of the product that ``_combine`` 
 and a query sees the keys of its own chunk only; pages of earlier chunks go back.  ``distance_bias``: a number a head;
 that slope times the distance i - j comes off the scores, after scale and cap.
 
+``conv``: a short causal convolution over time on every channel of q, k and v, directly behind the projections
+(``parts.conv`` adds one to a norm's rows; this one stands alone): y_t = sum_j w[:, j] * u_(t - n + 1 + j) with n taps and
+zeros before the first token.  A request's last n - 1 projected rows are its state, float32, a side entry of the mixer.
+``norm_over="projection"``: q, and k, are each divided by ONE root mean square over all their heads; the weights then have
+the projections' sizes.  ``null_sink``: every head's sink has the score 0 (a one in the denominator), without a tensor.
+``gate_name``: head h's result is multiplied by sigmoid(W_g x)_h before the output projection; the gate's matrix rides in
+the q|k|v product and the attention kernels apply it to the unrounded result.
+``own_kv=False``: the layer has no keys and values of its own; it reads the rows that another layer's call has cached
+(``cache_window``: how many positions that entry keeps, at least this mixer's window), with its own queries and mask.
+
 A mixer that stands beside others reads a share of ONE input product and leaves its rows for ONE output product:
 ``in_matrix`` / ``out_matrix`` are the matrices it wants there, ``mix`` is what lies between them.
 """
@@ -43,7 +53,7 @@ from __future__ import annotations
 import torch
 
 from tokasaurus_b200.kernels import ops
-from tokasaurus_b200.parts.base import Mixer, PagedCacheNeed, WeightSpec
+from tokasaurus_b200.parts.base import Mixer, PagedCacheNeed, StateNeed, WeightSpec
 
 
 class SinkAttention(Mixer):
@@ -56,8 +66,11 @@ class SinkAttention(Mixer):
                  rotary=None, rotary_pairs: bool = True, values_are_keys: bool = False,
                  head_scale_name: str | None = None, head_bias_name: str | None = None, weights: str = "softmax",
                  keep_first: int = 0, maps: int = 1, extra_names: tuple[tuple[str, int], ...] = (),
-                 chunk: int | None = None, distance_bias=None):
-        """``extra_names``: (tensor name, rows) of matrices [rows, width] appended to the q|k|v product."""
+                 chunk: int | None = None, distance_bias=None, conv: tuple[int, tuple[str, str, str]] | None = None,
+                 norm_over: str = "head", null_sink: bool = False, gate_name: str | None = None, own_kv: bool = True,
+                 cache_window: int | None | str = "same"):
+        """``extra_names``: (tensor name, rows) of matrices [rows, width] appended to the q|k|v product.  ``conv``: (taps, the tensor
+        names of q's, k's and v's taps [channels, taps])."""
         if n_heads % n_kv_heads:
             raise ValueError(f"n_heads={n_heads} is not a multiple of n_kv_heads={n_kv_heads}")
         if weights not in ("softmax", "sigmoid"):
@@ -76,6 +89,28 @@ class SinkAttention(Mixer):
             raise ValueError("a chunk or a sliding window, not both")
         if distance_bias is not None and (len(distance_bias) != n_heads or maps != 1):
             raise ValueError(f"{len(distance_bias)} distance slopes for {n_heads} heads of {maps} maps")
+        if norm_over not in ("head", "projection"):
+            raise ValueError(f"a norm of q and k is over a 'head' or the 'projection', not {norm_over!r}")
+        if norm_over == "projection" and (not unit_norm or qk_norm_names is None):
+            raise ValueError("a norm over the projection comes with its weights")
+        if conv is not None and (conv[0] < 1 or bias_names is not None or values_are_keys or norm_over == "projection"):
+            raise ValueError("a convolution has at least one tap; with biases, values that are the keys, or a norm over the "
+                             "projection it is not built")
+        if null_sink and (sink_name is not None or weights == "sigmoid"):
+            raise ValueError("a sink of score 0 takes the place of a learned one, in a softmax")
+        if gate_name is not None and maps != 1:
+            raise ValueError("an output gate within the attention needs one map a head")
+        if gate_name is not None:
+            extra_names = tuple(extra_names) + ((gate_name, n_heads),)
+        self.gated, self.null_sink, self.own_kv = gate_name is not None, bool(null_sink), bool(own_kv)
+        self.whole_norm = norm_over == "projection"
+        self.taps, self.conv_names = (int(conv[0]), tuple(conv[1])) if conv is not None else (0, None)
+        self.conv_w: torch.Tensor | None = None
+        if chunk and cache_window != "same":
+            raise ValueError("a chunk's keys are kept as long as the chunk")
+        if cache_window != "same" and cache_window is not None and (not window or window > cache_window):
+            raise ValueError(f"a window of {window} positions cannot be read from a cache entry that keeps {cache_window}")
+        self.cache_window = cache_window
         self.chunk = int(chunk) if chunk else None
         self.distance_bias = tuple(float(x) for x in distance_bias) if distance_bias is not None else None
         self.head_slope: torch.Tensor | None = None
@@ -94,48 +129,80 @@ class SinkAttention(Mixer):
         self.norm_eps, self.unit_norm = float(norm_eps), bool(unit_norm)
         self.names = (q_name, k_name, v_name, o_name)
         self.sink_name, self.bias_names, self.out_bias_name = sink_name, bias_names, out_bias_name
-        self.defines = ops.sink_attention_defines(dim, vdim, self.sigmoid, self.maps, self.distance_bias is not None)
+        self.defines = ops.sink_attention_defines(dim, vdim, self.sigmoid, self.maps, self.distance_bias is not None, self.taps)
         self.sinks = self.qkv_bias = self.out_bias = None
 
     def weight_specs(self):
         q, k, v, o = self.names
         H, G, d, e = self.n_heads, self.n_kv_heads, self.dim, self.vdim
         M = self.maps
-        specs = [WeightSpec(q, (H * M * d, self.width)), WeightSpec(k, (G * M * d, self.width)), WeightSpec(o, (self.width, H * e))]
+        own = self.own_kv
+        specs = [WeightSpec(q, (H * M * d, self.width)), WeightSpec(o, (self.width, H * e))]
         specs += [WeightSpec(n, (rows, self.width)) for n, rows in self.extra_names]
-        if not self.values_are_keys:
+        if own:
+            specs.append(WeightSpec(k, (G * M * d, self.width)))
+        if own and not self.values_are_keys:
             specs.append(WeightSpec(v, (G * e, self.width)))
         if self.qk_norm_names is not None:
-            specs += [WeightSpec(n, (d,), role="vector") for n in self.qk_norm_names]
+            sizes = (H * M * d, G * M * d) if self.whole_norm else (d, d)
+            specs += [WeightSpec(n, (c,), role="vector") for n, c in list(zip(self.qk_norm_names, sizes))[:2 if own else 1]]
+        if self.conv_names is not None:
+            specs += [WeightSpec(n, (c, self.taps), role="vector")
+                      for n, c in list(zip(self.conv_names, (H * M * d, G * M * d, G * e)))[:3 if own else 1]]
         specs += [WeightSpec(n, (H * M,), role="vector") for n in (self.head_scale_name, self.head_bias_name) if n is not None]
         if self.bias_names is not None:
             specs += [WeightSpec(n, (rows,), role="vector")
-                      for n, rows in zip(self.bias_names, (H * d, G * d) if self.values_are_keys else (H * M * d, G * M * d, G * e))]
+                      for n, rows in zip(self._own_biases(), (H * M * d, G * M * d, G * e))]
         if self.out_bias_name is not None:
             specs.append(WeightSpec(self.out_bias_name, (self.width,), role="vector"))
         if self.sink_name is not None:
             specs.append(WeightSpec(self.sink_name, (H * M,), role="vector"))
         return tuple(specs)
 
+    def _own_biases(self):
+        """The names of the biases on what the mixer projects itself."""
+        return self.bias_names[:(2 if self.values_are_keys else 3) if self.own_kv else 1]
+
     def kernel_modules(self, dtype):
         return (("attention_sink.cu", self.defines),)
 
+    def _conv_columns(self) -> int:
+        H, G, M = self.n_heads, self.n_kv_heads, self.maps
+        return H * M * self.dim + (G * (M * self.dim + self.vdim) if self.own_kv else 0)
+
+    def side_needs(self):
+        if self.taps < 2:
+            return {}
+        return {"conv": StateNeed(((self.taps - 1) * self._conv_columns(),), "float32")}
+
     def cache_need(self):
-        return PagedCacheNeed(self.n_kv_heads, self.maps * self.dim + self.vdim, self.chunk or self.window, planes=1,
+        window = self.window if self.cache_window == "same" else self.cache_window
+        return PagedCacheNeed(self.n_kv_heads, self.maps * self.dim + self.vdim, self.chunk or window, planes=1,
                               keep_first=self.keep_first, chunked=self.chunk is not None)
 
     def bind(self, weights, rt) -> None:
         q, k, v, o = self.names
-        self.w_qkv = torch.cat([weights[q], weights[k]] + ([] if self.values_are_keys else [weights[v]])
-                               + [weights[n] for n, _ in self.extra_names], dim=0).contiguous()
+        stack = [weights[q]]
+        if self.own_kv:
+            stack += [weights[k]] + ([] if self.values_are_keys else [weights[v]])
         # where the extra matrices' results start in a row of the product
-        self.extra_off = self.w_qkv.shape[0] - sum(rows for _, rows in self.extra_names)
+        self.extra_off = sum(w.shape[0] for w in stack)
+        stack += [weights[n] for n, _ in self.extra_names]
+        self.gate_off = sum(w.shape[0] for w in stack) - self.n_heads  # (the gate's matrix is the last)
+        odd = -sum(w.shape[0] for w in stack) % 8
+        if self.gated and odd:  # the product's rows stay whole 16-byte pieces
+            stack.append(torch.zeros((odd, self.width), dtype=stack[0].dtype, device=stack[0].device))
+        self.w_qkv = torch.cat(stack, dim=0).contiguous()
         self.w_o = weights[o].contiguous()
         if self.bias_names is not None:
-            names = self.bias_names[:2] if self.values_are_keys else self.bias_names
-            self.qkv_bias = torch.cat([weights[n].float() for n in names]).contiguous()
+            self.qkv_bias = torch.cat([weights[n].float() for n in self._own_biases()]).contiguous()
         if self.qk_norm_names is not None:
-            self.qk_norm_w = torch.stack([weights[n].float() for n in self.qk_norm_names]).contiguous()
+            # (a mixer without keys of its own: the second weight is never read)
+            names = self.qk_norm_names if self.own_kv else self.qk_norm_names[:1] * (1 if self.whole_norm else 2)
+            join = torch.cat if self.whole_norm else torch.stack
+            self.qk_norm_w = join([weights[n].float() for n in names]).contiguous()
+        if self.conv_names is not None:
+            self.conv_w = torch.cat([weights[n].float() for n in self.conv_names[:3 if self.own_kv else 1]], dim=0).contiguous()
         if self.rotary is not None and self.rotary.rotary_dim > 0:
             self.rot_freq = self.rotary.inv_freq64().to(rt.device)
         if self.distance_bias is not None:
@@ -148,6 +215,8 @@ class SinkAttention(Mixer):
             self.out_bias = weights[self.out_bias_name].contiguous()
         if self.sink_name is not None:
             self.sinks = weights[self.sink_name].contiguous()
+        elif self.null_sink:
+            self.sinks = torch.zeros((self.n_heads * self.maps,), dtype=torch.float32, device=rt.device)
 
     def _combine(self, ctx, attn, qkv, out_rows):
         """What goes into the output projection, from the attention's result ``attn`` ([rows, heads * maps * vdim]; with
@@ -165,26 +234,35 @@ class SinkAttention(Mixer):
         """The matrices live on in a wider product."""
         self.w_qkv = self.w_o = None
 
-    def forward(self, ctx, h, cache, out_rows=None):
+    def forward(self, ctx, h, cache, out_rows=None, side=None):
         qkv = ops.linear(h, self.w_qkv, out_dtype=torch.float32)
-        return ops.linear_out_f32(self.mix(ctx, qkv, cache, h.dtype, out_rows), self.w_o, ctx.status)
+        return ops.linear_out_f32(self.mix(ctx, qkv, cache, h.dtype, out_rows, side=side), self.w_o, ctx.status)
 
-    def mix(self, ctx, qkv, cache, dtype, out_rows=None, out=None, out_scale: float = 1.0):
+    def mix(self, ctx, qkv, cache, dtype, out_rows=None, out=None, out_scale: float = 1.0, side=None):
         """From the float32 product ``qkv`` of all tokens (a column slice will do) to what the output product reads, times
         ``out_scale``, in ``dtype``.  ``out`` (one map, all rows): where it goes, a column slice of a wider tensor."""
         H, G, d, e, M = self.n_heads, self.n_kv_heads, self.dim, self.vdim, self.maps
         T, dev = qkv.shape[0], qkv.device
         tables = ctx.tables[cache.group]
         q = torch.empty((T, H * M * d), dtype=dtype, device=dev)
-        ops.sink_attn_prep(qkv, self.qkv_bias, self.unit_norm, self.norm_eps, q, cache.k, ctx.positions, ctx.token_seq,
-                           tables.indptr, tables.page_ids, H, G, d, e, cache.page_size, cache.writable, ctx.status,
-                           norm_w=self.qk_norm_w, rot_freq=self.rot_freq,
-                           rot_dims=self.rotary.rotary_dim if self.rot_freq is not None else 0,
-                           rot_pairs=self.rotary_pairs, values_are_keys=self.values_are_keys, sigmoid=self.sigmoid, maps=M,
-                           distance=self.head_slope is not None)
+        prep = dict(norm_w=self.qk_norm_w, rot_freq=self.rot_freq, rot_pairs=self.rotary_pairs,
+                    rot_dims=self.rotary.rotary_dim if self.rot_freq is not None else 0, maps=M, own_kv=self.own_kv,
+                    sigmoid=self.sigmoid, distance=self.head_slope is not None)
+        if self.taps:
+            state = side["conv"] if self.taps > 1 else None
+            ops.sink_attn_conv_prep(qkv, self.conv_w, state.state if state is not None else None, self.unit_norm,
+                                    self.norm_eps, q, cache.k, ctx.positions, ctx.token_seq, ctx.seq_slot, ctx.seq_q_start,
+                                    ctx.seq_q_len, ctx.n_seqs, not ctx.single_token_step, tables.indptr, tables.page_ids, H, G,
+                                    d, e, cache.page_size, cache.writable, state is not None and state.writable, ctx.status,
+                                    **prep)
+        else:
+            ops.sink_attn_prep(qkv, self.qkv_bias, self.unit_norm, self.norm_eps, q, cache.k, ctx.positions, ctx.token_seq,
+                               tables.indptr, tables.page_ids, H, G, d, e, cache.page_size, cache.writable, ctx.status,
+                               values_are_keys=self.values_are_keys, whole_norm=self.whole_norm, **prep)
         out_dtype = dtype if M == 1 else torch.float32  # several maps' outputs stay unrounded for what combines them
         options = dict(head_scale=self.head_scale, head_bias=self.head_bias, sigmoid=self.sigmoid, maps=M,
-                       keep_first=self.keep_first, chunk=self.chunk, head_slope=self.head_slope, out_scale=out_scale)
+                       keep_first=self.keep_first, chunk=self.chunk, head_slope=self.head_slope, out_scale=out_scale,
+                       gate=qkv[:, self.gate_off:self.gate_off + H] if self.gated else None, taps=self.taps)
         if ops.can_use_attn_sink_tc(dtype, d, e, M):
             # bfloat16: every token on the tensor cores (single tokens and portions by a kernel each); wanted rows are
             # cut out afterwards

@@ -39,7 +39,10 @@ def random_tensors(specs: Iterable[WeightSpec], seed: int, std: float = 0.02, no
             continue
         if any(d < 0 for d in s.shape):  # a size that only a weight file knows: random weights take 16
             s = WeightSpec(s.name, tuple(16 if d < 0 else d for d in s.shape), s.role, s.keep_32bit)
-        if s.role == "table":
+        if s.role == "table" and s.below:
+            keys = torch.rand((*s.shape[:-1], s.below), generator=g, device=device)
+            out[s.name] = keys.argsort(dim=-1)[..., :s.shape[-1]].to(torch.int32).contiguous()
+        elif s.role == "table":
             out[s.name] = torch.randint(0, 2**15, s.shape, generator=g, dtype=torch.int32, device=device)
         elif s.role == "vector":
             if norm_init == "ones":
