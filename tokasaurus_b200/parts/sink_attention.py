@@ -137,10 +137,11 @@ class SinkAttention(Mixer):
         H, G, d, e = self.n_heads, self.n_kv_heads, self.dim, self.vdim
         M = self.maps
         own = self.own_kv
-        specs = [WeightSpec(q, (H * M * d, self.width)), WeightSpec(o, (self.width, H * e))]
-        specs += [WeightSpec(n, (rows, self.width)) for n, rows in self.extra_names]
+        specs = [WeightSpec(q, (H * M * d, self.width))]
         if own:
             specs.append(WeightSpec(k, (G * M * d, self.width)))
+        specs.append(WeightSpec(o, (self.width, H * e)))
+        specs += [WeightSpec(n, (rows, self.width)) for n, rows in self.extra_names]
         if own and not self.values_are_keys:
             specs.append(WeightSpec(v, (G * e, self.width)))
         if self.qk_norm_names is not None:
