@@ -2,7 +2,7 @@
 random weights (the metric and configuration of BASELINE.json's configs[2]).
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 2|3|4]
-    python bench.py --design sozurax|daborax|verozen|bibalix|safupel   (another workload, see run_design; the default workload and its output line are unchanged)
+    python bench.py --design sozurax|daborax|verozen|bibalix|safupel|deletar   (another workload, see run_design; the default workload and its output line are unchanged)
 
 Prints ONE JSON line.  ``value``: decoded tokens a second at batch 8, each request holding a
 2,048-token prompt in the cache, timed on the device with CUDA events around K decode steps
@@ -160,7 +160,7 @@ def prefill_flops(m: dict, T: int, rows: int = 1) -> float:
     return linear + attention
 
 
-TIMED_OPS = ("real_gated_recurrence", "memory_gates", "memory_norm", "act_rows", "diff_combine", "head_sigmoid_gate", "moe_logits", "sum_group_norm", "gelu_gate_rows", "gla_gates", "rotate_scale", "linear_out_f32", "scaled_norm_add", "cast_rows", "add_sinusoid", "clamped_glu", "gated_group_norm", "ssm_prep", "decay_walk",
+TIMED_OPS = ("norm_add_norm", "sink_attn_conv_prep", "moe_table", "soft_cap", "real_gated_recurrence", "memory_gates", "memory_norm", "act_rows", "diff_combine", "head_sigmoid_gate", "moe_logits", "sum_group_norm", "gelu_gate_rows", "gla_gates", "rotate_scale", "linear_out_f32", "scaled_norm_add", "cast_rows", "add_sinusoid", "clamped_glu", "gated_group_norm", "ssm_prep", "decay_walk",
              "sink_attn_prep", "attn_sink", "attn_sink_tc", "silu_cols", "gemm_tcgen05_clamped", "add_layernorm", "add_layernorm_conv1", "short_conv", "polynorm", "gated_recurrence", "latent_prep",
              "rotate_pairs", "latent_attn", "moe_route", "moe_order", "moe_gather", "moe_gemm", "moe_combine",
              "gemm_tcgen05_grouped", "embed_gather", "add_rmsnorm", "rope_kv_write", "rope_kv_write_partials", "linear_decode", "linear_smallm",
@@ -756,6 +756,33 @@ def safupel_configs(name: str) -> dict:
     return dict(safupel=saf, daborax=daborax_configs(name)["daborax"], verozen=verozen_configs(name)["verozen"])
 
 
+def deletar_configs(name: str) -> dict:
+    """Layer sizes for ``--design deletar``: two sizes that resemble a real model's layers, each as a Deletar decoder
+    (attention behind a short convolution with a dense feed-forward, attention normed over the projection with the keys for
+    values, attention with a one in the denominator, a reader of that layer's rows, these three with experts chosen by a
+    table; norms ahead of and behind every sublayer) and as the closest existing model, a Daborax decoder of attention
+    layers only (the same attention kernels, heads, window and capped scores, norms on the sublayers' outputs, a dense
+    feed-forward) at the same width, depth, vocabulary and head sizes; the like of its routed experts (ungated, grouped
+    products) is the Verozen decoder's."""
+    sizes = dict(w2048=dict(width=2048, heads=16, kv=4, ff=8192, experts=16, top=4, expert_ff=2048, shared_ff=2048),
+                 w4096=dict(width=4096, heads=32, kv=8, ff=14336, experts=16, top=4, expert_ff=3584, shared_ff=3584))
+    z = sizes[name]
+    W = z["width"]
+    dense = dict(kind="dense", ff=z["ff"])
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"]), router=dict(experts=z["experts"], top=z["top"]), shared=dict(ff=z["shared_ff"]))
+    att = dict(heads=z["heads"], kv_heads=z["kv"], dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024))
+    rot = dict(base=10000.0, dims=64, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))
+    third = dict(att, softcap=30.0, rot=rot)
+    dele = dict(architecture="Deletar", vocab=32000, width=W, norm=dict(eps=1e-6), embedding=dict(scale=1.0), logit_softcap=30.0,
+                layers=[dict(type="attention", mixer=dict(att, conv=4, rot=dict(base=250000.0, dims=64)), mlp=dense),
+                        dict(type="attention_2", mixer=dict(att, softcap=30.0, rot=dict(base=10000.0, dims=128)), mlp=moe),
+                        dict(type="attention_3", mixer=third, mlp=moe),
+                        dict(type="attention_3", mixer=dict(third, kv_from=2), mlp=moe)])
+    dab = dict(architecture="Daborax", vocab=32000, width=W, norm=dict(eps=1e-6), embedding=dict(scale=1.0), residual_mult=0.5,
+               layers=[dict(type="attention", mixer=dict(att, softcap=30.0), mlp=dict(dense, limit=7.0)) for _ in range(4)])
+    return dict(deletar=dele, daborax=dab, verozen=verozen_configs(name)["verozen"])
+
+
 def design_configs(name: str) -> dict:
     """Layer sizes for ``--design sozurax``: two sizes that resemble a real model's layers, each as a Sozurax decoder
     (a recurrent layer with a dense feed-forward, a latent-attention layer with routed experts, a second recurrent
@@ -785,7 +812,7 @@ def design_configs(name: str) -> dict:
 
 
 def run_design(args) -> dict:
-    """``--design sozurax|daborax|verozen|bibalix|safupel``: prefill (one 2,048-token prompt in one step) and decode (batch 8 and 64, prompts of
+    """``--design sozurax|daborax|verozen|bibalix|safupel|deletar``: prefill (one 2,048-token prompt in one step) and decode (batch 8 and 64, prompts of
     2,048 tokens in the cache) of that decoder at two layer sizes beside the closest existing decoder of equal size, random weights,
     bfloat16, with the CUDA-event time of each kind of kernel in one prefill step and one decode step of both."""
     import numpy as np
@@ -800,7 +827,7 @@ def run_design(args) -> dict:
     prompt_len, page_size = 2048, 16
     out = dict(design=args.design, dtype="bf16", data="synthetic", peaks=dict(peaks, source=peak_src), sizes={})
     configs_of = dict(daborax=daborax_configs, sozurax=design_configs, verozen=verozen_configs,
-                      bibalix=bibalix_configs, safupel=safupel_configs)[args.design]
+                      bibalix=bibalix_configs, safupel=safupel_configs, deletar=deletar_configs)[args.design]
     for size in ("w2048", "w4096"):
         res = {}
         for arch, cfg in configs_of(size).items():
@@ -815,7 +842,7 @@ def run_design(args) -> dict:
                 # forget gates lower bounds below one, so that tokens spread over the experts and states stay bounded
                 if isinstance(b.mixer, GatedLinearRecurrence):
                     b.mixer.lower.uniform_(0.0, 0.9, generator=g)
-                if isinstance(getattr(b, "ffn", None), RoutedExperts):
+                if isinstance(getattr(b, "ffn", None), RoutedExperts) and b.ffn.router_w is not None:
                     b.ffn.router_w.normal_(0.0, 1.0, generator=g)
                 if getattr(b.mixer, "lam", None) is not None:
                     b.mixer.lam.fill_(0.5)  # (vectors of ones would make the two maps' factor a difference of overflows)
@@ -913,7 +940,7 @@ def main() -> int:
     ap.add_argument("--config", type=int, default=2, choices=[2, 3, 4],
                     help="2: the headline metric (default); 3 and 4: the further workloads, see run_further")
     ap.add_argument("--design-arch", default=None, help="with --design: only this arm (the design's name or 'llama')")
-    ap.add_argument("--design", default=None, choices=["sozurax", "daborax", "verozen", "bibalix", "safupel"],
+    ap.add_argument("--design", default=None, choices=["sozurax", "daborax", "verozen", "bibalix", "safupel", "deletar"],
                     help="instead of the headline workload: this design's prefill and decode at two layer sizes beside "
                          "the closest existing decoder of equal size (see run_design)")
     args = ap.parse_args()

@@ -592,6 +592,71 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
   }
 }
 
+__device__ __forceinline__ float4 vec4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 vec4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const uint32_t*>(&a);
+  u.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+__device__ __forceinline__ float4 fma4(float w, float4 v, float4 a) {
+  return make_float4(fmaf(w, v.x, a.x), fmaf(w, v.y, a.y), fmaf(w, v.z, a.z), fmaf(w, v.w, a.w));
+}
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+// The same sums in the same order, four values a thread and the loads of four outputs (or slices) in flight: with one at a
+// time, rows of few tokens waited for memory once a value (eight tokens of width 4,096 with eight slices: 36 us).
+template <typename T, typename TY>
+__global__ void moe_combine_vec_kernel(const TY* __restrict__ y, const int* __restrict__ place_of,
+                                       const float* __restrict__ top_w, const T* __restrict__ shared_t,
+                                       const float* __restrict__ shared_slices, int n_slices, long long slice_stride,
+                                       T* __restrict__ out, int H, int top, const float* __restrict__ shared_gate) {
+  trigger_dependents();
+  grid_dependency_wait();
+  const int t = blockIdx.y;
+  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i >= H) return;
+  const float sg = shared_gate != nullptr ? 1.f / (1.f + expf(-shared_gate[t])) : 1.f;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 acc = zero;
+  for (int k0 = 0; k0 < top; k0 += 4) {
+    float4 v[4];
+    float w[4];
+    int p[4];
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const size_t pair = (size_t)t * top + k0 + j;
+      p[j] = k0 + j < top ? place_of[pair] : -1;
+      w[j] = top_w != nullptr && k0 + j < top ? top_w[pair] : 1.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; j++) v[j] = p[j] >= 0 ? vec4(y + (size_t)p[j] * H + i) : zero;
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+      if (p[j] >= 0) acc = fma4(w[j], v[j], acc);
+  }
+  float4 sh = shared_gate == nullptr ? acc : zero;  // with a gate the shared part is added up by itself
+  if (shared_t != nullptr) sh = add4(sh, vec4(shared_t + (size_t)t * H + i));
+  for (int s0 = 0; s0 < n_slices; s0 += 4) {
+    float4 q[4];
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+      q[j] = s0 + j < n_slices ? vec4(shared_slices + (size_t)(s0 + j) * slice_stride + (size_t)t * H + i) : zero;
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+      if (s0 + j < n_slices) sh = add4(sh, q[j]);
+  }
+  put4(out + (size_t)t * H + i, shared_gate == nullptr ? sh : fma4(sg, sh, acc));
+}
+
 template <typename T>
 int route_launch(const void* h, const float* wr, const float* br, const int* token_seq, int* top_idx, float* top_w,
                  float* logits, int n_tokens, int H, int E, int top, int over_all, float scale, cudaStream_t st) {
@@ -645,6 +710,13 @@ int combine_launch(const void* y, const int* place_of, const float* top_w, const
                    const float* shared_slices, int n_slices, long long slice_stride, void* out, int n_tokens, int H,
                    int top, const float* shared_gate, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
+  const uintptr_t all = ((uintptr_t)y) | ((uintptr_t)shared_t) | ((uintptr_t)shared_slices) | ((uintptr_t)out);
+  if ((H & 3) == 0 && (slice_stride & 3) == 0 && (all & 15) == 0 && n_tokens <= 65535) {
+    const int threads = H >= 1024 ? 256 : 64;
+    return launch_pdl(moe_combine_vec_kernel<T, TY>, dim3((H / 4 + threads - 1) / threads, n_tokens), dim3(threads), 0, st,
+                      (const TY*)y, place_of, top_w, (const T*)shared_t, shared_slices, n_slices, slice_stride, (T*)out, H,
+                      top, shared_gate);
+  }
   return launch_pdl(moe_combine_kernel<T, TY>, dim3(n_tokens), dim3(H >= 1024 ? 256 : 128), 0, st, (const TY*)y, place_of, top_w,
                     (const T*)shared_t, shared_slices, n_slices, slice_stride, (T*)out, H, top, shared_gate);
 }
